@@ -7,7 +7,8 @@ crates/pagedllm/src/blocks.rs:296-430).  Here layers whose mixers ask for the
 same kind of cache (all keys, or a window of them; the same kv heads and head
 size) form a group with pages, an allocator and tables of its own; a window
 group gives pages back as soon as the window has passed them, but for the pages
-of the first tokens that its mixers keep seeing (``keep_first``).  Mixers that ask
+of the first tokens that its mixers keep seeing (``keep_first``), and a chunk group
+those of the chunks before the current one.  Mixers that ask
 for a ``StateNeed`` get a slot of fixed size per request instead.
 
 One page holds ``page_size`` tokens of every layer of its group.  How a page
@@ -27,7 +28,16 @@ from ..errors import CacheError
 from ..parts.base import CompositeNeed, PagedNeed, StateNeed
 from .allocator import BlockAllocator, block_hash
 
-FREED = -1  # a table entry whose page was given back (window groups only)
+FREED = -1  # a table entry whose page was given back (groups whose queries read back a bounded way only)
+
+
+def _leaves(need, path: tuple):
+    """(path, need) of every piece of a possibly nested CompositeNeed."""
+    if isinstance(need, CompositeNeed):
+        for j, part in enumerate(need.parts):
+            yield from _leaves(part, path + (j,))
+    else:
+        yield path, need
 
 
 class BlockTable:
@@ -83,12 +93,16 @@ class CacheGroup:
     allocator: BlockAllocator
     page_size: int
     pool: Optional[torch.Tensor] = None  # need.pool_shape(entries, pages, page_size)
-    # per cache of the group, whose it is: the schedule entry, or (entry, part) for a part of a mixer made of several
+    # per cache of the group, whose it is: the schedule entry, or (entry, part, ...) for a piece of a CompositeNeed
     cells: List[object] = field(default_factory=list)
 
     @property
     def window(self) -> Optional[int]:
         return self.need.window if self.need.kind == "window" else None
+
+    @property
+    def chunk(self) -> int:
+        return self.need.chunk if self.need.kind == "chunk" else 0
 
     @property
     def kept_pages(self) -> int:
@@ -121,17 +135,16 @@ class CacheManager:
         self.page_size, self.num_pages, self.max_requests = page_size, num_pages, max_requests
         self.dtype, self.device = dtype, device
         self.groups: List[CacheGroup] = []
-        # A cell is what one need gets: schedule entry i, or (i, j) for part j of an entry whose mixer is made of several
-        # (a CompositeNeed).
+        # A cell is what one need gets: schedule entry i, or (i, j, ...) for a piece of an entry's CompositeNeed.
         self._entry_group: Dict[object, Tuple[int, int]] = {}  # cell -> (group, index in group)
         self._state_entries: Dict[object, StateNeed] = {}
-        self._composite: Dict[int, int] = {}                   # entry -> how many parts
+        self._composite: Dict[int, CompositeNeed] = {}         # entry -> what it asks for
         by_key: Dict[tuple, int] = {}
         cells = []
         for i, need in enumerate(needs):
             if isinstance(need, CompositeNeed):
-                self._composite[i] = len(need.parts)
-                cells += [((i, j), i, part) for j, part in enumerate(need.parts)]
+                self._composite[i] = need
+                cells += [(path, i, part) for path, part in _leaves(need, (i,))]
             else:
                 cells.append((i, i, need))
         for cell, i, need in cells:
@@ -156,7 +169,7 @@ class CacheManager:
         # Sharing rests on pages that never change and are never dropped while held:
         # true for groups that keep every key, not for windows or state.
         self.prefix_cache = bool(prefix_cache) and bool(self.groups) and not self._state_entries \
-            and all(g.window is None for g in self.groups)
+            and all(g.need.reach() is None for g in self.groups)
         if allocate_device:
             for g in self.groups:
                 g.pool = torch.zeros(g.need.pool_shape(len(g.entries), num_pages, page_size),
@@ -176,8 +189,13 @@ class CacheManager:
         for cell, t in self._state.items():
             by_cell[cell] = t
         out: List[object] = [by_cell.get(i) for i in range(self._n_entries)]
-        for i, n in self._composite.items():
-            out[i] = tuple(by_cell.get((i, j)) for j in range(n))
+
+        def assembled(need, path):
+            if isinstance(need, CompositeNeed):
+                return tuple(assembled(part, path + (j,)) for j, part in enumerate(need.parts))
+            return by_cell.get(path)
+        for i, need in self._composite.items():
+            out[i] = assembled(need, (i,))
         return out
 
     def bytes_per_token(self) -> int:
@@ -231,13 +249,14 @@ class CacheManager:
 
     def pages_for(self, tokens: int, step_tokens: Optional[int] = None) -> int:
         """Pages a request of ``tokens`` tokens holds at its largest, in the group
-        that needs most.  A window group holds the window plus what one step adds."""
+        that needs most.  A window (or chunk) group holds the window (or chunk) plus what one step adds."""
         most = 0
         for g in self.groups:
-            if g.window is None:
+            reach = g.need.reach()
+            if reach is None:
                 n = -(-tokens // self.page_size)
             else:
-                span = min(tokens, g.window + (step_tokens or tokens))
+                span = min(tokens, reach + (step_tokens or tokens))
                 n = min(-(-tokens // self.page_size), -(-span // self.page_size) + 1 + g.kept_pages)
             most = max(most, n)
         return most
@@ -310,7 +329,7 @@ class CacheManager:
     def commit(self, request_id, count: int, history: Optional[Sequence[int]] = None) -> None:
         """Record that ``count`` tokens were written.  Names the pages that became
         full (``history`` = every token of the request so far) and gives back the
-        pages a window has passed."""
+        pages a window has passed, or those of finished chunks."""
         rc = self.get(request_id)
         if not rc.tables:
             rc._tokens += count
@@ -328,10 +347,10 @@ class CacheManager:
                     name = block_hash(t.hashes[-1] if t.hashes else None, chunk)
                     t.hashes.append(name)
                     g.allocator.publish(t.blocks[i], name)
-            if g.window is not None:
-                # The next query sits at position t.tokens or later and sees keys
-                # from t.tokens - window + 1 on: pages wholly before that are done.
-                first_needed = max(0, t.tokens - g.window + 1)
+            if g.need.reach() is not None:
+                # The next query sits at position t.tokens or later: pages wholly before the
+                # first key that it reads are done.
+                first_needed = g.need.first_read(t.tokens)
                 while (t.first_live + 1) * self.page_size <= first_needed:
                     b = t.blocks[t.first_live]
                     if b >= 0 and t.first_live >= g.kept_pages:      # (the pages of the kept first tokens stay)
@@ -340,7 +359,7 @@ class CacheManager:
                     t.first_live += 1
 
     def set_prefix_cache(self, enabled: bool) -> None:
-        enabled = bool(enabled) and bool(self.groups) and not self._state_entries and all(g.window is None for g in self.groups)
+        enabled = bool(enabled) and bool(self.groups) and not self._state_entries and all(g.need.reach() is None for g in self.groups)
         self.prefix_cache = enabled
         if not enabled:
             for g in self.groups:

@@ -3,7 +3,8 @@
 //
 // For the query at position p of head h (kv head h / group), over cached tokens j:
 //     s_j   = cap * tanh(scale * (q . k_j) / cap)          (cap = 0: s_j = scale * (q . k_j))
-//     seen  = j <= p and (p - j < window or j < keep_first) (window = 0: every j <= p)
+//     seen  = j <= p and (p - j < window or j < keep_first) (window = 0: every j <= p; with chunk > 0 only the j of p's own
+//             chunk: floor(j / chunk) = floor(p / chunk))
 //     out   = sum_seen exp(s_j) v_j / (exp(sink_h) + sum_seen exp(s_j))
 // The sink is a learned logit per head that takes weight and gives no value (sinks null: none).
 // Scores, the softmax and the weighted sum are float whatever the cache's dtype.
@@ -24,6 +25,11 @@ enum : int { KID_ATT_SINK = 70 };
 #define SINK_BK 32         // keys per tile
 #define SINK_MAX_ROWS 16   // query rows (token x head of the group) per CTA, one warp each
 #define SINK_MAX_D 256     // largest key size and largest value size
+
+// the first key that position `pos` sees (the kept first tokens aside)
+__device__ __forceinline__ int sink_first_seen(int pos, int window, int chunk) {
+    return window > 0 ? pos - window + 1 : chunk > 0 ? pos - pos % chunk : 0;
+}
 
 struct SinkWork { int seg, q_token0, q_count, q_pos0, kv_begin, kv_end, part_slot, split; };
 
@@ -110,7 +116,7 @@ __global__ void attention_sink_kernel(const T* q,                 // [tokens, nh
                                       const int* __restrict__ n_work_ptr, T* __restrict__ out,   // [tokens, nh, dv]
                                       float* __restrict__ part_o, float* __restrict__ part_ml,
                                       const float* __restrict__ sinks, int nh, int nkv, int dk, int dv, int page_size, int n_pages,
-                                      int table_width, int window, int keep_first, float scale, float cap, int heads_per_cta,
+                                      int table_width, int window, int keep_first, int chunk, float scale, float cap, int heads_per_cta,
                                       int* status) {
     pdl_launch_dependents();
     pdl_wait(KID_ATT_SINK);
@@ -134,7 +140,7 @@ __global__ void attention_sink_kernel(const T* q,                 // [tokens, nh
     const bool active = warp < rows;
     const int tq = active ? warp / n_heads : 0;
     const int head = active ? head0 + warp % n_heads : head0;
-    const int pos = w.q_pos0 + tq;
+    const int pos = w.q_pos0 + tq, first_seen = sink_first_seen(pos, window, chunk);
     if (active) {
         const T* qr = q + ((size_t)(w.q_token0 + tq) * nh + head) * dk;
         for (int e = lane; e < dk; e += 32) q_s[warp * dk + e] = to_f32(qr[e]);
@@ -198,7 +204,7 @@ __global__ void attention_sink_kernel(const T* q,                 // [tokens, nh
             __syncthreads();
             if (!active) continue;
             const int j = kv0 + lane;
-            const bool visible = j < r_end && j <= pos && (window <= 0 || pos - j < window || j < keep_first);
+            const bool visible = j < r_end && j <= pos && (j >= first_seen || j < keep_first);
             if (!__any_sync(0xffffffffu, visible)) continue;
             float s = 0.f;
             {
@@ -263,9 +269,9 @@ __global__ void attention_sink_kernel(const T* q,                 // [tokens, nh
 PLLM_EXPORT int pllm_attention_sink(int dtype, const void* q, const void* kv_pool, const int* block_tables, const int* work,
                                     const int* n_work_ptr, int max_work, void* out, float* part_o, float* part_ml,
                                     const float* sinks, int nh, int nkv, int dk, int dv, int page_size, int n_pages, int table_width,
-                                    int window, int keep_first, float scale, float cap, int* status, cudaStream_t stream) {
+                                    int window, int keep_first, int chunk, float scale, float cap, int* status, cudaStream_t stream) {
     if (max_work <= 0) return PLLM_OK;
-    if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || window < 0 || keep_first < 0) return PLLM_ERR_SIZE;
+    if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || window < 0 || keep_first < 0 || chunk < 0 || (chunk && (window || keep_first))) return PLLM_ERR_SIZE;
     if (dk <= 0 || dv <= 0) return PLLM_ERR_SIZE;
     if (dk > SINK_MAX_D || dv > SINK_MAX_D) return PLLM_ERR_LIMIT;
     const int group = nh / nkv;
@@ -278,7 +284,7 @@ PLLM_EXPORT int pllm_attention_sink(int dtype, const void* q, const void* kv_poo
         dim3 grid(max_work, nkv * gparts);
         launch_chained(attention_sink_kernel<T>, grid, dim3(SINK_MAX_ROWS * 32), smem, stream, (const T*)q, (const T*)kv_pool,
                        block_tables, (const SinkWork*)work, n_work_ptr, (T*)out, part_o, part_ml, sinks, nh, nkv, dk, dv, page_size,
-                       n_pages, table_width, window, keep_first, scale, cap, heads_per_cta, status);
+                       n_pages, table_width, window, keep_first, chunk, scale, cap, heads_per_cta, status);
     });
     return launch_status();
 }
@@ -329,7 +335,7 @@ __global__ void __launch_bounds__(128, (DK + DV <= 192) ? 4 : 3) attention_sink_
                                                                  bf16* __restrict__ out, float* __restrict__ part_o,
                                                                  float* __restrict__ part_ml, const float* __restrict__ sinks, int nh,
                                                                  int nkv, int page_size, int n_pages, int table_width, int window,
-                                                                 int keep_first, float scale, float cap, int heads_per_cta, int* status) {
+                                                                 int keep_first, int chunk, float scale, float cap, int heads_per_cta, int* status) {
     constexpr int QS = DK + SMMA_PAD, KS = DK + SMMA_PAD, VS = DV + SMMA_PAD;      // row strides in elements
     extern __shared__ __align__(16) unsigned char sink_smem[];
     bf16* q_s = reinterpret_cast<bf16*>(sink_smem);            // [SMMA_ROWS][QS]
@@ -370,10 +376,12 @@ __global__ void __launch_bounds__(128, (DK + DV <= 192) ? 4 : 3) attention_sink_
     const int r0 = row_base + g, r1 = r0 + 8;
     const int pos0 = w.q_pos0 + (r0 < rows ? r0 / n_heads : 0), pos1 = w.q_pos0 + (r1 < rows ? r1 / n_heads : 0);
     const bool live0 = r0 < rows, live1 = r1 < rows;
+    const int seen0 = sink_first_seen(pos0, window, chunk), seen1 = sink_first_seen(pos1, window, chunk);
     // positions of the warp's rows, for skipping tiles: rows warp*16 .. warp*16+15 that exist
     const int wr_lo = row_base, wr_hi = min(rows, row_base + 16) - 1;
     const bool warp_live = wr_lo < rows;
     const int wpos_lo = w.q_pos0 + wr_lo / n_heads, wpos_hi = w.q_pos0 + (warp_live ? wr_hi / n_heads : 0);
+    const int wseen_lo = sink_first_seen(wpos_lo, window, chunk);
 
     float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
     float o[DV / 8][4];
@@ -428,7 +436,7 @@ __global__ void __launch_bounds__(128, (DK + DV <= 192) ? 4 : 3) attention_sink_
             const int t_lo = ksplit ? kv0 + warp * 16 : kv0;
             const int t_hi = min(ksplit ? t_lo + 16 : kv0 + SMMA_BK, r_end) - 1;
             bool any = warp_live && t_lo <= wpos_hi && t_lo < r_end;
-            if (any && window > 0) any = t_hi > wpos_lo - window || t_lo < keep_first;
+            if (any) any = t_hi >= wseen_lo || t_lo < keep_first;
             if (any) {
                 float sc[SMMA_BK / 8][4];
 #pragma unroll
@@ -454,7 +462,7 @@ __global__ void __launch_bounds__(128, (DK + DV <= 192) ? 4 : 3) attention_sink_
                         const int key = kv0 + j * 8 + t4 * 2 + (e & 1);
                         const int pos = e < 2 ? pos0 : pos1;
                         const bool live = e < 2 ? live0 : live1;
-                        const bool seen = live && key < r_end && key <= pos && (window <= 0 || pos - key < window || key < keep_first);
+                        const bool seen = live && key < r_end && key <= pos && (key >= (e < 2 ? seen0 : seen1) || key < keep_first);
                         float v = sc[j][e] * scale;
                         // tanh(x) = 1 - 2 / (exp(2x) + 1) with the fast exponential and division: its absolute error (1e-7) is far
                         // below what the bfloat16 operands leave in the score
@@ -591,7 +599,7 @@ PLLM_EXPORT int pllm_attention_sink_mma_tile_tokens(int nh, int nkv) {
 template <int DK, int DV>
 static int launch_sink_mma(const void* q, const void* kv_pool, const int* block_tables, const int* work, const int* n_work_ptr, int max_work,
                            void* out, float* part_o, float* part_ml, const float* sinks, int nh, int nkv, int page_size, int n_pages,
-                           int table_width, int window, int keep_first, float scale, float cap, int* status, cudaStream_t stream) {
+                           int table_width, int window, int keep_first, int chunk, float scale, float cap, int* status, cudaStream_t stream) {
     const int group = nh / nkv;
     const int heads_per_cta = group < SMMA_ROWS ? group : SMMA_ROWS;
     const int gparts = (group + heads_per_cta - 1) / heads_per_cta;
@@ -603,21 +611,21 @@ static int launch_sink_mma(const void* q, const void* kv_pool, const int* block_
     cudaFuncSetAttribute(attention_sink_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_chained(attention_sink_mma_kernel<DK, DV>, dim3(max_work, nkv * gparts), dim3(128), smem, stream, (const bf16*)q,
                    (const bf16*)kv_pool, block_tables, (const SinkWork*)work, n_work_ptr, (bf16*)out, part_o, part_ml, sinks, nh, nkv,
-                   page_size, n_pages, table_width, window, keep_first, scale, cap, heads_per_cta, status);
+                   page_size, n_pages, table_width, window, keep_first, chunk, scale, cap, heads_per_cta, status);
     return launch_status();
 }
 
 PLLM_EXPORT int pllm_attention_sink_mma(const void* q, const void* kv_pool, const int* block_tables, const int* work,
                                         const int* n_work_ptr, int max_work, void* out, float* part_o, float* part_ml,
                                         const float* sinks, int nh, int nkv, int dk, int dv, int page_size, int n_pages, int table_width,
-                                        int window, int keep_first, float scale, float cap, int* status, cudaStream_t stream) {
+                                        int window, int keep_first, int chunk, float scale, float cap, int* status, cudaStream_t stream) {
     if (max_work <= 0) return PLLM_OK;
-    if (!pllm_attention_sink_mma_supports(PLLM_BF16, nh, nkv, dk, dv) || page_size <= 0 || window < 0 || keep_first < 0) return PLLM_ERR_SIZE;
+    if (!pllm_attention_sink_mma_supports(PLLM_BF16, nh, nkv, dk, dv) || page_size <= 0 || window < 0 || keep_first < 0 || chunk < 0 || (chunk && (window || keep_first))) return PLLM_ERR_SIZE;
     if (((uintptr_t)q | (uintptr_t)kv_pool) & 15) return PLLM_ERR_ALIGN;
 #define SINK_MMA_CASE(A, B)                                                                                                     \
     if (dk == A && dv == B)                                                                                                     \
         return launch_sink_mma<A, B>(q, kv_pool, block_tables, work, n_work_ptr, max_work, out, part_o, part_ml, sinks, nh, nkv, \
-                                     page_size, n_pages, table_width, window, keep_first, scale, cap, status, stream);
+                                     page_size, n_pages, table_width, window, keep_first, chunk, scale, cap, status, stream);
     SINK_MMA_CASE(32, 32) SINK_MMA_CASE(32, 64) SINK_MMA_CASE(32, 128)
     SINK_MMA_CASE(64, 32) SINK_MMA_CASE(64, 64) SINK_MMA_CASE(64, 128)
     SINK_MMA_CASE(128, 32) SINK_MMA_CASE(128, 64) SINK_MMA_CASE(128, 128)

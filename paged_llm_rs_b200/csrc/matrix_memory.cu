@@ -21,21 +21,13 @@
 // meet: what a token's output is does not depend on how the columns are shared out among CTAs, and on where a prompt was
 // cut only by the rounding of the delta rule's pairs of tokens.  Other threads of the CTA fetch the tokens ahead of the
 // recurrence.
-#include "common.cuh"
-
-enum : int { KID_MATRIX_MEMORY = 100 };
+#include "matrix_memory.cuh"
 
 #define MM_CHUNK 32            // tokens fetched at a time (fewer where keys are so long that shared memory would not hold them)
 #define MM_CHUNK_SMALL 8       // ... in a step of decoded tokens
 #define MM_CONV_TOKENS 64      // tokens a CTA of the convolution
 #define MM_MAX_TAPS 16
 
-struct MMSegment { int first, count, before, slot; };
-
-__device__ __forceinline__ float mm_silu(float z) { return z / (1.0f + expf(-z)); }
-__device__ __forceinline__ float mm_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float mm_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
-__device__ __forceinline__ float mm_logsigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float mm_parts_sum(float v, int parts) {
     if (parts > 16) v += __shfl_xor_sync(0xffffffffu, v, 16);
     if (parts > 8) v += __shfl_xor_sync(0xffffffffu, v, 8);
@@ -95,23 +87,6 @@ __global__ void __launch_bounds__(128) mm_conv_silu_kernel(const T* u, int u_wid
 #define MM_LOADERS_SMALL 32      // ... in a step of decoded tokens
 
 __device__ __forceinline__ void mm_loader_barrier(int loaders) { asm volatile("bar.sync 1, %0;\n" ::"r"(loaders) : "memory"); }
-
-template <typename T> struct MMVec;
-template <> struct MMVec<float> { static constexpr int N = 4; };
-template <> struct MMVec<bf16> { static constexpr int N = 8; };
-
-// 16 bytes at p (on a 16-byte boundary), times scale, as floats to shared memory (dst on a 16-byte boundary)
-__device__ __forceinline__ void mm_fetch16(const float* p, float* dst, float scale) {
-    const float4 v = *reinterpret_cast<const float4*>(p);
-    *reinterpret_cast<float4*>(dst) = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
-}
-__device__ __forceinline__ void mm_fetch16(const bf16* p, float* dst, float scale) {
-    const uint4 r = *reinterpret_cast<const uint4*>(p);
-    *reinterpret_cast<float4*>(dst) = make_float4(__uint_as_float(r.x << 16) * scale, __uint_as_float(r.x & 0xffff0000u) * scale,
-                                                  __uint_as_float(r.y << 16) * scale, __uint_as_float(r.y & 0xffff0000u) * scale);
-    *reinterpret_cast<float4*>(dst + 4) = make_float4(__uint_as_float(r.z << 16) * scale, __uint_as_float(r.z & 0xffff0000u) * scale,
-                                                      __uint_as_float(r.w << 16) * scale, __uint_as_float(r.w & 0xffff0000u) * scale);
-}
 
 // grid (segments, heads, slices of e).  c: [tokens, channels] float, q at 0 (G d), k at G d, v at 2 G d (H e).
 // ba: [tokens, 2 H] float, b_raw | a_raw.  u (the projection, for the convolution's state): [tokens, u_width] with the
@@ -664,34 +639,6 @@ __global__ void __launch_bounds__(128) mlstm_store_nm_kernel(const float* __rest
     if (threadIdx.x == 0) slot[(size_t)H * d * E + (size_t)H * d + h] = nm[d];
 }
 
-// A warp a (token, head): o / rms(o) * gain * act(gate).  y float [tokens, H e]; gate: [tokens, g_stride] of the compute dtype;
-// gain_per_head: the gain has H e entries, else e entries shared by the heads; kind 0 sigmoid, 1 silu.  With dn ([tokens, H, 2]:
-// the normaliser's product with the query, exp(-m)) y holds numerators, and o = y / (max(|n . q|, exp(-m)) + 1e-6).
-template <typename T>
-__global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* y, const float* __restrict__ dn, const T* gate, int g_stride,
-                                                             const float* __restrict__ gain, T* __restrict__ out, long long n_rows,
-                                                             int H, int E, int gain_per_head, int kind, float eps) {
-    pdl_launch_dependents();
-    pdl_wait(KID_MATRIX_MEMORY);
-    const int lane = threadIdx.x & 31;
-    const long long r = blockIdx.x * (long long)(blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (r >= n_rows) return;
-    const long long t = r / H;
-    const int h = (int)(r % H);
-    const float* yr = y + r * E;
-    const T* gr = gate + t * g_stride + (size_t)h * E;
-    const float over = dn ? fmaxf(fabsf(dn[r * 2]), dn[r * 2 + 1]) + 1e-6f : 1.0f;
-    float ss = 0.f;
-    for (int i = lane; i < E; i += 32) { const float v = yr[i] / over; ss += v * v; }
-    ss = warp_sum(ss);
-    const float inv = 1.0f / sqrtf(ss / (float)E + eps);
-    for (int i = lane; i < E; i += 32) {
-        const float z = to_f32(gr[i]);
-        const float sg = mm_sigmoid(z);
-        out[r * E + i] = from_f32<T>(yr[i] / over * inv * gain[gain_per_head ? h * E + i : i] * (kind == 1 ? z * sg : sg));
-    }
-}
-
 struct MMShape { int parts, npt, Ps, slices, workers, threads, chunk; size_t smem; };
 
 // The delta rule: PARTS threads a column so that a thread holds at most 16 rows (32 for the longest keys), columns a CTA so
@@ -746,14 +693,6 @@ static inline int mlstm_shape(int n_segs, int H, int d, int E, int max_segment_t
     out->chunk = chunk;
     out->smem = smem_of(chunk);
     return (out->smem > 200 * 1024 || out->threads > MM_SCAN_THREADS) ? PLLM_ERR_LIMIT : PLLM_OK;
-}
-
-template <typename T>
-static void launch_head_norm_gate(const float* y, const float* dn, const void* gate, int g_stride, const float* gain, void* out, int n_tokens, int H, int E,
-                                  int gain_per_head, int kind, float eps, cudaStream_t stream) {
-    const long long rows = (long long)n_tokens * H;
-    launch_chained(head_norm_gate_kernel<T>, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, stream, y, dn, (const T*)gate, g_stride, gain,
-                   (T*)out, rows, H, E, gain_per_head, kind, eps);
 }
 
 #define MM_NPT_DISPATCH(npt, CALL) do { if ((npt) == 4) { constexpr int NPT = 4; CALL; } else if ((npt) == 8) { constexpr int NPT = 8; CALL; } \

@@ -1,0 +1,67 @@
+// What the recurrences with a matrix of state a head share: a step's segments, loads of 16 bytes as floats, and the head
+// norm with its gate behind a recurrence.
+#pragma once
+
+#include "common.cuh"
+
+enum : int { KID_MATRIX_MEMORY = 100 };
+
+struct MMSegment { int first, count, before, slot; };
+
+__device__ __forceinline__ float mm_silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float mm_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float mm_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float mm_logsigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+template <typename T> struct MMVec;
+template <> struct MMVec<float> { static constexpr int N = 4; };
+template <> struct MMVec<bf16> { static constexpr int N = 8; };
+
+// 16 bytes at p (on a 16-byte boundary), times scale, as floats to shared memory (dst on a 16-byte boundary)
+__device__ __forceinline__ void mm_fetch16(const float* p, float* dst, float scale) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    *reinterpret_cast<float4*>(dst) = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+}
+__device__ __forceinline__ void mm_fetch16(const bf16* p, float* dst, float scale) {
+    const uint4 r = *reinterpret_cast<const uint4*>(p);
+    *reinterpret_cast<float4*>(dst) = make_float4(__uint_as_float(r.x << 16) * scale, __uint_as_float(r.x & 0xffff0000u) * scale,
+                                                  __uint_as_float(r.y << 16) * scale, __uint_as_float(r.y & 0xffff0000u) * scale);
+    *reinterpret_cast<float4*>(dst + 4) = make_float4(__uint_as_float(r.z << 16) * scale, __uint_as_float(r.z & 0xffff0000u) * scale,
+                                                      __uint_as_float(r.w << 16) * scale, __uint_as_float(r.w & 0xffff0000u) * scale);
+}
+
+// A warp a (token, head): o / rms(o) * gain * act(gate).  y float [tokens, H e]; gate: [tokens, g_stride] of the compute dtype;
+// gain_per_head: the gain has H e entries, else e entries shared by the heads (null: no gain); kind 0 sigmoid, 1 silu.  With dn ([tokens, H, 2]:
+// the normaliser's product with the query, exp(-m)) y holds numerators, and o = y / (max(|n . q|, exp(-m)) + 1e-6).
+template <typename T>
+__global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* y, const float* __restrict__ dn, const T* gate, int g_stride,
+                                                             const float* __restrict__ gain, T* __restrict__ out, long long n_rows,
+                                                             int H, int E, int gain_per_head, int kind, float eps) {
+    pdl_launch_dependents();
+    pdl_wait(KID_MATRIX_MEMORY);
+    const int lane = threadIdx.x & 31;
+    const long long r = blockIdx.x * (long long)(blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (r >= n_rows) return;
+    const long long t = r / H;
+    const int h = (int)(r % H);
+    const float* yr = y + r * E;
+    const T* gr = gate + t * g_stride + (size_t)h * E;
+    const float over = dn ? fmaxf(fabsf(dn[r * 2]), dn[r * 2 + 1]) + 1e-6f : 1.0f;
+    float ss = 0.f;
+    for (int i = lane; i < E; i += 32) { const float v = yr[i] / over; ss += v * v; }
+    ss = warp_sum(ss);
+    const float inv = 1.0f / sqrtf(ss / (float)E + eps);
+    for (int i = lane; i < E; i += 32) {
+        const float z = to_f32(gr[i]);
+        const float sg = mm_sigmoid(z);
+        out[r * E + i] = from_f32<T>(yr[i] / over * inv * (gain ? gain[gain_per_head ? h * E + i : i] : 1.0f) * (kind == 1 ? z * sg : sg));
+    }
+}
+
+template <typename T>
+static void launch_head_norm_gate(const float* y, const float* dn, const void* gate, int g_stride, const float* gain, void* out, int n_tokens, int H, int E,
+                                  int gain_per_head, int kind, float eps, cudaStream_t stream) {
+    const long long rows = (long long)n_tokens * H;
+    launch_chained(head_norm_gate_kernel<T>, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, stream, y, dn, (const T*)gate, g_stride, gain,
+                   (T*)out, rows, H, E, gain_per_head, kind, eps);
+}
+

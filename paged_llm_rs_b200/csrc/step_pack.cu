@@ -17,6 +17,7 @@ struct PllmGroupPack {
     const int* const* tables;   // [n] each request's block table of this group (int32; -1: page given back)
     const int* table_len;       // [n] entries in each
     int window;                 // 0: every key stays
+    int chunk;                  // > 0 (and no window): a query reads its own chunk of this many positions only
     int ctas_per_item;          // CTAs the attention kernel launches per work item
     int max_work, max_red, max_parts;                                    // capacities of the captured step
     int plans;                  // 0: the group's mixers take no attention work items (the offsets of work and red are unused)
@@ -91,7 +92,7 @@ PLLM_EXPORT int pllm_pack_decode_step(int* out, int out_len, int n, const int* t
         for (int i = 0; i < n; i++) {
             const int p0 = positions[i];
             const int kv_end = p0 + 1;
-            const int kv_begin = g.window > 0 ? (p0 - (g.window - 1) > 0 ? p0 - (g.window - 1) : 0) : 0;
+            const int kv_begin = g.window > 0 ? (p0 - (g.window - 1) > 0 ? p0 - (g.window - 1) : 0) : (g.chunk > 0 ? p0 - p0 % g.chunk : 0);
             const int keys = kv_end - kv_begin;
             int splits = 1;
             if (want > 1) {

@@ -240,14 +240,14 @@ class _DecodeGraph:
 def group_plans(cache: CacheManager, mixer_of, page_size: int) -> List[Optional[GroupPlanConfig]]:
     """Per cache group how its attention is cut into work items: what its mixers wish (those of one group alike; a group
     whose mixers wish for nothing gets tables and slots only).  ``mixer_of(cell)`` gives the mixer a cache of the group
-    belongs to (``CacheGroup.cells``: a schedule entry, or (entry, part) for a part of a mixer made of several)."""
+    belongs to (``CacheGroup.cells``: a schedule entry, or (entry, part, ...) for a piece of a CompositeNeed)."""
     plans = []
     for g in cache.groups:
         wishes = {mixer_of(cell).plan_wish(page_size) for cell in g.cells}
         if len(wishes) != 1:
             raise ConfigError(f"the mixers that share a cache group wish for different attention plans: {sorted(map(str, wishes))}")
         w = wishes.pop()
-        plans.append(None if w is None else GroupPlanConfig(w.tile_tokens, w.ctas_per_item, g.window, w.heads, w.head_dim))
+        plans.append(None if w is None else GroupPlanConfig(w.tile_tokens, w.ctas_per_item, g.window, w.heads, w.head_dim, g.chunk))
     return plans
 
 
@@ -304,10 +304,9 @@ class ModelRunner:
         self.last_launches = 0    # kernels of this library the last step launched
 
     def _mixer_of(self, cell):
-        """The mixer that a cache of a group belongs to: a schedule entry's, or part j of it for a cell (entry, j)."""
-        entry, part = cell if isinstance(cell, tuple) else (cell, None)
-        mixer = self.model.blocks[self.model.schedule[entry].layer].mixer
-        return mixer if part is None else mixer.parts[part]
+        """The mixer that a cache of a group belongs to: a schedule entry's, or a part of it for a cell (entry, part, ...)."""
+        entry, path = (cell[0], cell[1:]) if isinstance(cell, tuple) else (cell, ())
+        return self.model.blocks[self.model.schedule[entry].layer].owner(path)
 
     # -- the step ----------------------------------------------------------------------
     def step(self, entries: Sequence[StepEntry], check: bool = True, trace: Optional[dict] = None) -> torch.Tensor:

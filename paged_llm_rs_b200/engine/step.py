@@ -46,6 +46,7 @@ class GroupPlanConfig:
     window: Optional[int]
     heads: int = 1        # partial results of split items are [rows, heads, head_dim]
     head_dim: int = 1
+    chunk: int = 0        # a query reads its own chunk of this many tokens only (0: no chunks)
 
 
 @dataclass
@@ -156,12 +157,12 @@ class StepPacker:
             if plan is None:        # the group's mixers read tables and slots only
                 group_parts.append((slots, tables, None, None, 0, 0, 0, W))
                 continue
-            # groups that cut their work alike (same tile, window, CTAs an item) share one plan
-            key = (plan.tile_tokens, plan.window, plan.ctas_per_item)
+            # groups that cut their work alike (same tile, window, chunk, CTAs an item) share one plan
+            key = (plan.tile_tokens, plan.window, plan.ctas_per_item, plan.chunk)
             if key not in planned:
                 planned[key] = attention_plan.plan_attention(
                     [(t0, n, p0) for (t0, n, p0, _) in segs], plan.tile_tokens, plan.window, plan.ctas_per_item,
-                    self.target_ctas)
+                    self.target_ctas, chunk=plan.chunk)
             work, red, parts = planned[key]
             mw, mr, mp = (work_caps[gi] if work_caps else (len(work), len(red), parts))
             if len(work) > mw or len(red) > mr or parts > mp:
@@ -257,7 +258,7 @@ class StepPacker:
 class _GroupPack(ctypes.Structure):
     """csrc/step_pack.cu: PllmGroupPack."""
     _fields_ = [("tables", ctypes.POINTER(ctypes.c_void_p)), ("table_len", ctypes.POINTER(ctypes.c_int)),
-                ("window", ctypes.c_int), ("ctas_per_item", ctypes.c_int),
+                ("window", ctypes.c_int), ("chunk", ctypes.c_int), ("ctas_per_item", ctypes.c_int),
                 ("max_work", ctypes.c_int), ("max_red", ctypes.c_int), ("max_parts", ctypes.c_int),
                 ("plans", ctypes.c_int),
                 ("off_slots", ctypes.c_int), ("off_tables", ctypes.c_int), ("off_n_work", ctypes.c_int),
@@ -302,7 +303,7 @@ class NativeDecodePacker:
             g.table_len = ctypes.cast(lens, ctypes.POINTER(ctypes.c_int))
             g.plans = 0 if plan is None else 1
             if plan is not None:
-                g.window, g.ctas_per_item = int(plan.window or 0), plan.ctas_per_item
+                g.window, g.chunk, g.ctas_per_item = int(plan.window or 0), int(plan.chunk), plan.ctas_per_item
                 g.max_work, g.max_red, g.max_parts = work_caps[gi]
             for name in ("slots", "tables") + (("n_work", "n_red", "work", "red") if plan is not None else ()):
                 setattr(g, f"off_{name}", layout[f"g{gi}.{name}"][0])

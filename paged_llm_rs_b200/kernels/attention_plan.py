@@ -2,7 +2,7 @@
 
 A segment is the run of consecutive tokens one request brings to a step.  It is
 cut into tiles of at most ``tile_tokens`` query tokens; a tile attends over the
-keys from the start of its window (or 0) up to its last token.  When a step has
+keys from the start of its first token's window or chunk (or 0) up to its last token.  When a step has
 too few tiles to fill the GPU and a tile's key range is long (decoding, or a
 short portion late in a long prompt), the range is split and the splits are
 combined by the reduce kernel, always in the same order.
@@ -38,9 +38,9 @@ MULTI_MIN_SPLIT_KEYS = 2048
 def plan_attention(segments: Sequence[Tuple[int, int, int]], tile_tokens: int, window: Optional[int],
                    ctas_per_item: int, target_ctas: int,
                    min_split_keys: int = MIN_SPLIT_KEYS,
-                   multi_min_split_keys: int = MULTI_MIN_SPLIT_KEYS) -> Tuple[np.ndarray, np.ndarray, int]:
+                   multi_min_split_keys: int = MULTI_MIN_SPLIT_KEYS, chunk: int = 0) -> Tuple[np.ndarray, np.ndarray, int]:
     """segments: (first token index, token count, position of the first token) per
-    segment, in step order.  Returns (work [n, 8], red [m, 4], partial rows used)."""
+    segment, in step order; ``chunk``: a query reads keys of its own chunk of that many positions only.  Returns (work [n, 8], red [m, 4], partial rows used)."""
     seg_ids, q0s, qns, p0s = [], [], [], []
     if segments and all(c == 1 for _, c, _ in segments):
         # a decode step: one tile per segment, no per-segment array work
@@ -61,7 +61,7 @@ def plan_attention(segments: Sequence[Tuple[int, int, int]], tile_tokens: int, w
         return np.zeros((0, 8), np.int32), np.zeros((0, 4), np.int32), 0
     seg = np.concatenate(seg_ids); q0 = np.concatenate(q0s); qn = np.concatenate(qns); p0 = np.concatenate(p0s)
     kv_end = p0 + qn
-    kv_begin = np.maximum(0, p0 - (window - 1)) if window else np.zeros_like(p0)
+    kv_begin = np.maximum(0, p0 - (window - 1)) if window else (p0 - p0 % chunk if chunk else np.zeros_like(p0))
     n_tiles = len(seg)
     keys = kv_end - kv_begin
 

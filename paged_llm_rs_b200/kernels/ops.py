@@ -93,11 +93,11 @@ def lib():
         sig["pllm_add_scaled32"] = [c_int, P, P, c_float, c_ll, P]
         sig["pllm_scale32"] = [P, c_float, c_ll, P]
         sig["pllm_rope_mix_kv_write"] = [c_int, P, c_int, P, P, c_int, P, P, P, P, c_int, P] + [c_int] * 6 + [c_ll, P, P]
-        sig["pllm_attention_sink"] = [c_int, P, P, P, P, P, c_int, P, P, P, P] + [c_int] * 9 + [c_float, c_float, P, P]
+        sig["pllm_attention_sink"] = [c_int, P, P, P, P, P, c_int, P, P, P, P] + [c_int] * 10 + [c_float, c_float, P, P]
         sig["pllm_attention_sink_tile_tokens"] = [c_int, c_int]
         sig["pllm_attention_sink_mma_supports"] = [c_int] * 5
         sig["pllm_attention_sink_mma_tile_tokens"] = [c_int, c_int]
-        sig["pllm_attention_sink_mma"] = [P, P, P, P, P, c_int, P, P, P, P] + [c_int] * 9 + [c_float, c_float, P, P]
+        sig["pllm_attention_sink_mma"] = [P, P, P, P, P, c_int, P, P, P, P] + [c_int] * 10 + [c_float, c_float, P, P]
         sig["pllm_mamba2_mix"] = [c_int] + [P] * 8 + [c_int, c_int, P, c_ll, P, P, P] + [c_int] * 7 + [c_float, P]
         sig["pllm_pack_decode_step"] = [P, c_int, c_int, P, P, P, P, P] + [c_int] * 16 + [P, P]
         sig["pllm_sandwich_norm32"] = [c_int, P, P, P, P, P, P, P, c_int, c_int, c_float, P]
@@ -111,7 +111,14 @@ def lib():
         sig["pllm_latent_rope_write"] = [c_int, P, c_int, P, c_float, P, c_int, P, P, P, P, P, P, P] + [c_int] * 6 + [c_ll, P, P]
         sig["pllm_mlstm_mix"] = [c_int, P, c_int, P, P, P, c_float, P, P, c_int, c_int, P, c_ll, P, P, P, P] + [c_int] * 4 + [c_float, P]
         sig["pllm_delta_mix"] = [c_int, P, c_int, P, P, P, P, P, P, c_int, c_int, P, c_ll, P, P, P] + [c_int] * 6 + [c_float, P]
-        wide = {"pllm_mlstm_state_floats": [c_int] * 3, "pllm_delta_state_floats": [c_int] * 5}
+        sig["pllm_gated_sum_norm32"] = [c_int, P, P, c_int, c_float, P, c_int, c_float, P, c_int, P, P, c_int, P, c_int, P, P, P, P, P, P, P, P, P, P, P,
+                                        c_int, P, c_ll, P, c_int, c_int, c_float, P]
+        sig["pllm_poly_norm"] = [c_int, P, c_int, P, P, c_int, c_int, c_float, P]
+        sig["pllm_softcap32"] = [P, c_float, c_ll, P]
+        sig["pllm_linear_attention_mix"] = [c_int, P] + [c_int] * 5 + [c_float, c_float, c_int, P, P, P, P, P, c_int, c_float, P, P, c_int, c_int, P, c_ll,
+                                            P, P, P] + [c_int] * 4 + [c_float, P]
+        wide = {"pllm_linear_attention_state_floats": [c_int] * 3, "pllm_linear_attention_scratch_floats": [c_int] * 6,
+                "pllm_mlstm_state_floats": [c_int] * 3, "pllm_delta_state_floats": [c_int] * 5}
         for name, args in wide.items():
             fn = getattr(L, name)
             fn.argtypes = args
@@ -1048,10 +1055,10 @@ def attention_sink_ctas_per_item(num_heads: int, num_kv_heads: int, dtype: torch
 
 def attention_sink(q: torch.Tensor, kv_pool: torch.Tensor, block_tables: torch.Tensor, w, out: torch.Tensor,
                    sinks: Optional[torch.Tensor], num_heads: int, num_kv_heads: int, dk: int, dv: int, window: int, keep_first: int,
-                   scale: float, cap: float, status: torch.Tensor) -> torch.Tensor:
+                   scale: float, cap: float, status: torch.Tensor, chunk: int = 0) -> torch.Tensor:
     """Attention of the step's tokens over rows [k | v] of the paged pool [pages, kv_heads, page_size, dk + dv]:
     score = cap tanh(scale q.k / cap) (cap 0: uncapped); key j is seen from position p when j <= p and (p - j < window or
-    j < keep_first) (window 0: every j <= p); the softmax's denominator also holds exp(sinks[head]).  ``w`` is the group's
+    j < keep_first) (window 0: every j <= p, or with ``chunk`` those of p's own chunk); the softmax's denominator also holds exp(sinks[head]).  ``w`` is the group's
     ``AttentionWork``; then the reduction of split items.  q [T, heads, dk], out [T, heads, dv]."""
     work, n_work, max_work, red, n_red, max_red = w.work, w.n_work, w.max_work, w.red, w.n_red, w.max_red
     part_o, part_ml = w.part_o, w.part_ml
@@ -1075,12 +1082,12 @@ def attention_sink(q: torch.Tensor, kv_pool: torch.Tensor, block_tables: torch.T
     if attention_sink_uses_tensor_cores(q.dtype, num_heads, num_kv_heads, dk, dv):
         _check(L.pllm_attention_sink_mma(_ptr(q), _ptr(kv_pool), _ptr(block_tables), _ptr(work), _ptr(n_work), max_work, _ptr(out),
                                          _ptr(part_o), _ptr(part_ml), _ptr(sinks), num_heads, num_kv_heads, dk, dv, page_size, n_pages,
-                                         block_tables.shape[-1], int(window), int(keep_first), float(scale), float(cap), _ptr(status),
+                                         block_tables.shape[-1], int(window), int(keep_first), int(chunk), float(scale), float(cap), _ptr(status),
                                          _stream()), "attention_sink (mma)")
     else:
         _check(L.pllm_attention_sink(_code(q), _ptr(q), _ptr(kv_pool), _ptr(block_tables), _ptr(work), _ptr(n_work), max_work,
                                      _ptr(out), _ptr(part_o), _ptr(part_ml), _ptr(sinks), num_heads, num_kv_heads, dk, dv, page_size,
-                                     n_pages, block_tables.shape[-1], int(window), int(keep_first), float(scale), float(cap),
+                                     n_pages, block_tables.shape[-1], int(window), int(keep_first), int(chunk), float(scale), float(cap),
                                      _ptr(status), _stream()), "attention_sink")
     _check(L.pllm_attention_reduce(_code(q), _ptr(part_o), _ptr(part_ml), _ptr(red), _ptr(n_red), max_red, _ptr(out), num_heads, dv,
                                    1 if (w.many_splits and dv * 4 <= 1024) else 0, _stream()), "attention_reduce")
@@ -1450,3 +1457,132 @@ def latent_rope_write(down: Optional[torch.Tensor], gain: Optional[torch.Tensor]
                                         _ptr(positions), _ptr(inv_freq), T, heads, dim, rot_dim, int(rot), kv_rank, pool_rows,
                                         _ptr(status), _stream()), "latent_rope_write")
     return q_rows
+
+
+# ---- a float32 stream with gated sublayers side by side and a token shift (csrc/gated_stream.cu) ----------------------------
+
+def _cols(t: Optional[torch.Tensor], shape, dtype, what: str) -> int:
+    """The row stride of a [rows, width] tensor that may be a column range of a wider one (0: absent)."""
+    if t is None:
+        return 0
+    if not t.is_cuda or t.shape != shape or t.dtype != dtype or t.stride(1) != 1:
+        raise KernelError(f"{what} must be {tuple(shape)} of {dtype} on the GPU with unit inner stride")
+    return t.stride(0)
+
+
+def gated_sum_norm32(x: torch.Tensor, gain: torch.Tensor, out: torch.Tensor, eps: float, mixed=None, mixed_scale: float = 1.0, mixed2=None,
+                     mixed2_scale: float = 1.0, mixed_gate=None, mixed_bias=None, fed=None, fed_gate=None, fed_bias=None, embedded=None,
+                     vector=None, x_out=None, shift=None, shifted=None, segments=None, state=None, gain2=None, out2=None,
+                     rows=None) -> torch.Tensor:
+    """x' = x + sigmoid(mixed_gate + mixed_bias) (mixed_scale mixed + mixed2_scale mixed2) + sigmoid(fed_gate + fed_bias) fed
+    + embedded + vector (terms may be absent), float32, to ``x_out`` if given (x stays as it is); ``out`` = norm(x') gain;
+    ``shifted`` = h + (the token before's h - h) shift with h = norm(x') gain, the token before a segment's first from the
+    request's row of ``state`` [slots, width], which then takes the segment's last h; ``out2`` = norm(x') gain2.  With ``rows``
+    only those rows are formed and normed, into ``out``."""
+    _dev(x, gain, out, mixed_bias, fed_bias, embedded, vector, x_out, shift, shifted, segments, state, gain2, out2, rows)
+    for t, n in ((x, "x"), (gain, "gain"), (mixed_bias, "mixed_bias"), (fed_bias, "fed_bias"), (embedded, "embedded"), (vector, "vector"),
+                 (x_out, "x_out"), (shift, "shift"), (state, "state"), (gain2, "gain2")):
+        _f32(t, n)
+    _i32(rows, "rows")
+    T, W = x.shape
+    n = rows.numel() if rows is not None else T
+    strides = [_cols(t, (T, W), out.dtype, f"gated_sum_norm32: {name}") for t, name in
+               ((mixed, "mixed"), (mixed2, "mixed2"), (mixed_gate, "mixed_gate"), (fed, "fed"), (fed_gate, "fed_gate"))]
+    if out.shape != (n, W) or any(t is not None and t.numel() != W for t in (gain, gain2, mixed_bias, fed_bias, vector, shift)):
+        raise KernelError("gated_sum_norm32: out must be [rows, width], gains, biases, vector and shift of the stream's width")
+    if any(t is not None and t.shape != x.shape for t in (embedded, x_out)) or any(t is not None and (t.shape != x.shape or t.dtype != out.dtype)
+                                                                                  for t in (shifted, out2)):
+        raise KernelError("gated_sum_norm32: embedded, x_out, shifted and out2 must have x's shape, the latter two out's dtype")
+    if shifted is not None:
+        _segments_ok(segments, "gated_sum_norm32")
+        if state is None or state.dim() != 2 or state.shape[1] < W:
+            raise KernelError("gated_sum_norm32: the shift needs state slots of the stream's width")
+    _check(lib().pllm_gated_sum_norm32(
+        _code(out), _ptr(x), _ptr(mixed), strides[0], float(mixed_scale), _ptr(mixed2), strides[1], float(mixed2_scale), _ptr(mixed_gate), strides[2],
+        _ptr(mixed_bias), _ptr(fed), strides[3], _ptr(fed_gate), strides[4], _ptr(fed_bias), _ptr(embedded), _ptr(vector), _ptr(x_out), _ptr(gain),
+        _ptr(out), _ptr(shift), _ptr(shifted), _ptr(gain2), _ptr(out2), _ptr(segments), segments.shape[0] if segments is not None else 0,
+        _ptr(state), state.stride(0) if state is not None else 0, _ptr(rows), n, W, float(eps), _stream()), "gated_sum_norm32")
+    return out
+
+
+def poly_norm(u: torch.Tensor, coefficients: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """out = a N(u) + b N(u^2) + c N(u^3) + e row by row, N(z) = z / sqrt(mean(z^2) + eps); coefficients float32 [4];
+    ``u`` may be a column range of a wider tensor."""
+    _dev(coefficients, out)
+    _f32(coefficients, "coefficients")
+    stride = _cols(u, tuple(out.shape), out.dtype, "poly_norm: u")
+    if coefficients.numel() != 4:
+        raise KernelError("poly_norm: four coefficients")
+    _check(lib().pllm_poly_norm(_code(out), _ptr(u), stride, _ptr(coefficients), _ptr(out), out.shape[0], out.shape[1], float(eps), _stream()),
+           "poly_norm")
+    return out
+
+
+def softcap32(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x (float32, in place) = cap tanh(x / cap)."""
+    _dev(x)
+    _f32(x, "x")
+    if not cap > 0:
+        raise KernelError(f"softcap32: the cap must be positive, got {cap}")
+    _check(lib().pllm_softcap32(_ptr(x), float(cap), x.numel(), _stream()), "softcap32")
+    return x
+
+
+# ---- linear attention with decay (csrc/linear_attention.cu) ------------------------------------------------------------------
+
+def linear_attention_state_floats(heads: int, dim: int, vdim: int) -> int:
+    """Floats of a request's state slot: every head's matrix."""
+    return heads * dim * vdim
+
+
+def linear_attention_mix(u: torch.Tensor, q_off: int, k_off: int, v_off: int, gate_off: int, q_scale: float, k_scale: float, rot: int,
+                         inv_freq: Optional[torch.Tensor], decay: Optional[torch.Tensor], a1: Optional[torch.Tensor],
+                         a2: Optional[torch.Tensor], a_bias: Optional[torch.Tensor], tau: float, gain: Optional[torch.Tensor],
+                         segments: torch.Tensor, max_segment_tokens: int, state: torch.Tensor, out: torch.Tensor, heads: int, dim: int,
+                         vdim: int, eps: float) -> torch.Tensor:
+    """From a stacked projection ``u`` [T, width] (q and k [heads dim], v and the gate [heads vdim] at the given columns) to the
+    output projection's input [T, heads vdim]: q and k times their scales, turned on their first ``rot`` entries; per head
+    S <- diag(alpha) S + k v^T, o = S^T q over each segment's tokens from and into its state slot; each head over its root mean
+    square, the gain (vdim entries shared by the heads, or None), silu(gate).  alpha: ``decay`` (float32 [heads]), or, where
+    that is None, sigmoid(a2 a1 + a_bias)^(1 / tau) a key entry with a1 float32 [T, rank] and a2 [heads dim, rank].
+    ``max_segment_tokens`` bounds a segment's tokens (1: the form for decoded tokens)."""
+    _dev(u, inv_freq, decay, a1, a2, a_bias, gain, segments, state, out)
+    for t, n in ((inv_freq, "inv_freq"), (decay, "decay"), (a1, "a1"), (a_bias, "a_bias"), (gain, "gain"), (state, "state")):
+        _f32(t, n)
+    _segments_ok(segments, "linear_attention_mix")
+    T, width = u.shape
+    if max(q_off, k_off) + heads * dim > width or max(v_off, gate_off) + heads * vdim > width:
+        raise KernelError("linear_attention_mix: the projection is narrower than its parts")
+    if out.shape != (T, heads * vdim) or out.dtype != u.dtype:
+        raise KernelError("linear_attention_mix: out must be [T, heads vdim] of u's dtype")
+    if rot and (inv_freq is None or inv_freq.numel() * 2 != rot):
+        raise KernelError("linear_attention_mix: inv_freq must hold rot / 2 frequencies")
+    rank = 0
+    if decay is not None:
+        if decay.numel() != heads:
+            raise KernelError("linear_attention_mix: one decay a head")
+    else:
+        if a1 is None or a2 is None or a_bias is None or a1.dim() != 2 or not tau > 0:
+            raise KernelError("linear_attention_mix: decays a key entry need a1, a2, a bias and a positive tau")
+        rank = a1.shape[1]
+        if a1.shape[0] != T or a2.shape != (heads * dim, rank) or a2.dtype != u.dtype or a_bias.numel() != heads * dim:
+            raise KernelError("linear_attention_mix: a1 must be [T, rank], a2 [heads dim, rank] of u's dtype, the bias [heads dim]")
+    if gain is not None and gain.numel() != vdim:
+        raise KernelError("linear_attention_mix: a gain of vdim entries")
+    if state.dim() != 2 or state.shape[1] < heads * dim * vdim:
+        raise KernelError("linear_attention_mix: the state slots are too small")
+    longest = int(max_segment_tokens)
+    scratch = y_buf = None
+    launches = 1
+    if longest != 1:
+        floats = int(lib().pllm_linear_attention_scratch_floats(T, longest, heads, dim, vdim, 0 if decay is not None else 1))
+        scratch = torch.empty(floats, dtype=torch.float32, device=u.device) if floats else None
+        y_buf = torch.empty((T, heads * vdim), dtype=torch.float32, device=u.device)
+        alpha_only = 0 if decay is not None else -(-T * heads * dim // 4) * 4
+        launches = 2 + (decay is None) + (2 if floats > alpha_only else 0)
+    _check(lib().pllm_linear_attention_mix(
+        _code(u), _ptr(u), width, int(q_off), int(k_off), int(v_off), int(gate_off), float(q_scale), float(k_scale), int(rot), _ptr(inv_freq),
+        _ptr(decay), _ptr(a1), _ptr(a2), _ptr(a_bias), rank, 1.0 / float(tau) if decay is None else 1.0, _ptr(gain), _ptr(segments),
+        segments.shape[0], longest, _ptr(state), state.stride(0), _ptr(scratch), _ptr(y_buf), _ptr(out), T, heads, dim, vdim, float(eps),
+        _stream()), "linear_attention_mix", launches=launches)
+    return out

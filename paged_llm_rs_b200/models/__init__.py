@@ -3,3 +3,4 @@ from . import surelorn  # registers Surelorn
 from . import bumisun  # registers Bumisun
 from . import pamarax  # registers Pamarax
 from . import tebozen  # registers Tebozen
+from . import reperax  # registers Reperax

@@ -54,13 +54,25 @@ class Runtime:
 class PagedNeed:
     """Something kept for every token of a request, in pages that the cache manager hands out and
     takes back.  kind "full": everything stays until the request ends; "window": only the last
-    ``window`` tokens are ever read, so older pages are given back.  A need says how its pages lie
-    in memory; needs with equal ``group_key()`` share pages, an allocator and block tables.
+    ``window`` tokens are ever read, so older pages are given back; "chunk": a query reads only tokens of its own chunk
+    of ``chunk`` tokens (counted from the sequence's start), so the pages of earlier chunks are given back.  A need says
+    how its pages lie in memory; needs with equal ``group_key()`` share pages, an allocator and block tables.
     Every need has the fields ``kind``, ``window`` and ``dtype`` (None: the model's dtype).  A window need may also
     say ``keep_first``: the pages that hold a request's first ``keep_first`` tokens stay with it whatever the window
     has passed."""
 
     keep_first = 0
+    chunk = 0
+
+    def reach(self) -> Optional[int]:
+        """The most tokens, its own among them, that a query reads; None: all before it."""
+        return self.window if self.kind == "window" else self.chunk if self.kind == "chunk" else None
+
+    def first_read(self, position: int) -> int:
+        """The first position that a query at ``position`` or later reads (the kept first tokens aside)."""
+        if self.kind == "window":
+            return max(0, position - self.window + 1)
+        return position - position % self.chunk if self.kind == "chunk" else 0
 
     def group_key(self) -> tuple:
         raise NotImplementedError
@@ -108,7 +120,7 @@ class KVNeed(PagedNeed):
 class JoinedKVNeed(PagedNeed):
     """Paged keys and values whose sizes may differ, a token's key and value side by side in one row a kv head:
     a layer's rows as [pages, kv_heads, page_size, key_dim + value_dim].  With kind "window" only the last ``window``
-    tokens and the first ``keep_first`` are ever read."""
+    tokens and the first ``keep_first`` are ever read, with kind "chunk" only those of the query's chunk."""
 
     kind: str
     num_kv_heads: int
@@ -118,9 +130,10 @@ class JoinedKVNeed(PagedNeed):
     keep_first: int = 0
     group_size: int = 1          # query heads to a kv head (mixers that cut their attention alike share work items)
     dtype: Optional[torch.dtype] = None
+    chunk: int = 0
 
     def group_key(self) -> tuple:
-        return ("joined_kv", self.kind, self.window, self.keep_first, self.num_kv_heads, self.key_dim, self.value_dim,
+        return ("joined_kv", self.kind, self.window, self.keep_first, self.chunk, self.num_kv_heads, self.key_dim, self.value_dim,
                 self.group_size, self.dtype)
 
     def pool_shape(self, entries, pages, page_size):
@@ -170,8 +183,8 @@ class StateNeed:
 
 @dataclass(frozen=True)
 class CompositeNeed:
-    """What a mixer made of several mixers asks for: each part's need (a PagedNeed, a StateNeed or None), in the parts'
-    order.  The mixer is handed a tuple of what each part would have been handed alone."""
+    """What a mixer (or a block) made of several parts asks for: each part's need (a PagedNeed, a StateNeed, another
+    CompositeNeed or None), in the parts' order.  It is handed a tuple of what each part would have been handed alone."""
 
     parts: Tuple[Optional[object], ...]
 
@@ -328,9 +341,33 @@ class Block:
 
     kind = ""
     prefix = ""   # the layer's tensor prefix ("model.layers.3"), set by the decoder that builds it
+    keeps_stream = False   # True: the stream that forward() is given is not written to
 
-    def __init__(self, mixer: Mixer, feed_forward: FeedForward, norms: Dict[str, Norm]):
-        self.mixer, self.feed_forward, self.norms = mixer, feed_forward, norms
+    def __init__(self, mixer: Mixer, feed_forward: FeedForward, norms: Dict[str, Norm], extras: Optional[Dict[str, Part]] = None):
+        self.mixer, self.feed_forward, self.norms, self.extras = mixer, feed_forward, norms, extras or {}
+
+    def prepare(self) -> None:
+        """Called once when every part has its tensors: an arrangement may stack what its products share."""
+
+    def cache_need(self):
+        """What a run of the layer keeps: its mixer's need, unless the arrangement keeps something of its own beside it."""
+        return self.mixer.cache_need()
+
+    def owner(self, path: tuple):
+        """The part that a cache belongs to, given its path in the (nested) ``CompositeNeed`` of ``cache_need``."""
+        part = self.mixer
+        for j in path:
+            part = part.parts[j]
+        return part
+
+    def add_ahead(self, residual, handed_on, embedded, vector):
+        """Add the embedding's output (or None) and one vector for all tokens (or None) to the residual stream ahead of this
+        block, which a schedule entry may ask for; returns the pair that the block is then given.  What is pending is added
+        later, so the order does not matter to a stream that is a plain sum."""
+        for t in (embedded, vector):
+            if t is not None:
+                residual.add_(t.to(residual.dtype))
+        return residual, handed_on
 
     def forward(self, residual, delta, step: StepState, cache, writes_cache: bool):
         raise NotImplementedError
@@ -361,6 +398,7 @@ POSITION_ENCODINGS: Dict[str, type] = {}
 BLOCKS: Dict[str, type] = {}
 EMBEDDINGS: Dict[str, type] = {}
 HEADS: Dict[str, type] = {}
+EXTRAS: Dict[str, type] = {}       # what an arrangement needs beside mixer, feed-forward and norms (gates on results, ...)
 
 
 def _register(table: Dict[str, type], kind: str, cls: type, replace: bool) -> type:
@@ -378,6 +416,7 @@ def register_position_encoding(kind, cls, replace=False): return _register(POSIT
 def register_block(kind, cls, replace=False): return _register(BLOCKS, kind, cls, replace)
 def register_embedding(kind, cls, replace=False): return _register(EMBEDDINGS, kind, cls, replace)
 def register_head(kind, cls, replace=False): return _register(HEADS, kind, cls, replace)
+def register_extra(kind, cls, replace=False): return _register(EXTRAS, kind, cls, replace)
 
 
 def make(table: Dict[str, type], what: str, spec: PartSpec, rt: Runtime, **extra):

@@ -7,8 +7,11 @@ from __future__ import annotations
 
 import torch
 
+import torch
+
 from ..kernels import ops
-from .base import Block, register_block
+from .base import Block, CompositeNeed, register_block
+from .norm import PendingGated
 
 
 class PreNormResidualBlock(Block):
@@ -109,6 +112,65 @@ class SandwichStreamBlock(Block):
         return self.post_mixer(stream, a, step)
 
 
+class SideBySideGatedStreamBlock(Block):
+    """x + g1 * mixer(shift(norm1(x))) + g2 * ff(norm2(x)) on a float32 stream: both sublayers read the same x, each result is
+    multiplied by a gate of its normed input (g1 of norm1(x) ahead of the shift, g2 of norm2(x)), and the mixer's input is
+    shifted by a token.  Its norms are ``GatedStreamRMSNorm``s named "mixer" and "feed_forward"; its extras "mixer_gate",
+    "feed_forward_gate" (``ResidualGate``) and "shift" (``TokenShift``).  A layer may have no feed-forward.  What is handed on
+    beside the stream is all that is pending (``PendingGated``): ONE kernel adds it, norms the sum twice and shifts it.  The
+    stream that a block is given stays as it is; a run of the layer keeps what its mixer keeps and a row a request."""
+
+    keeps_stream = True
+
+    def __init__(self, mixer, feed_forward, norms, extras=None):
+        super().__init__(mixer, feed_forward, norms, extras)
+        self.shift, self.gate = self.extras["shift"], self.extras["mixer_gate"]
+        self.fed_gate = self.extras["feed_forward_gate"] if feed_forward is not None else None
+        self.w_fed = None
+
+    def prepare(self):
+        # the feed-forward's first product and its gate's read the same input: one product over both
+        if self.feed_forward is not None:
+            self.w_fed = torch.cat([self.feed_forward.w_first, self.fed_gate.weight], 0).contiguous()
+            n = self.feed_forward.w_first.shape[0]
+            self.feed_forward.w_first, self.fed_gate.weight = self.w_fed[:n], self.w_fed[n:]
+
+    def cache_need(self):
+        return CompositeNeed((self.mixer.cache_need(), self.shift.cache_need()))
+
+    def owner(self, path):
+        return super().owner(path[1:]) if path[:1] == (0,) else self.shift
+
+    def add_ahead(self, stream, pending, embedded, vector):
+        pending = pending or PendingGated()
+        pending.embedded, pending.vector = embedded, vector
+        return stream, pending
+
+    def forward(self, stream, pending, step, cache, writes_cache=True):
+        rt, norm1, norm2 = self.mixer.rt, self.norms["mixer"], self.norms["feed_forward"]
+        kept, last = cache
+        new = lambda: torch.empty(stream.shape, dtype=rt.dtype, device=stream.device)
+        h, shifted, h2 = new(), new(), new() if self.feed_forward is not None else None
+        x = torch.empty_like(stream) if pending is not None else None
+        ops.gated_sum_norm32(stream, norm1.gain, h, norm1.eps, x_out=x, shift=self.shift.mix, shifted=shifted, segments=step.segments,
+                             state=last, gain2=norm2.gain if h2 is not None else None, out2=h2,
+                             **(pending.arguments() if pending is not None else {}))
+        stream = stream if x is None else x
+        if hasattr(self.mixer, "forward_terms"):
+            terms = self.mixer.forward_terms(shifted, step, kept, writes_cache)
+        else:
+            terms = [(self.mixer.forward(shifted, step, kept, writes_cache), 1.0)]
+        out = PendingGated(terms, (self.gate.logits(h), self.gate.bias))
+        if h2 is not None:
+            u = ops.linear(h2, self.w_fed, status=rt.status)
+            n = self.feed_forward.w_first.shape[0]
+            out.fed, out.fed_gate = self.feed_forward.forward_rest(u[:, :n], step), (u[:, n:], self.fed_gate.bias)
+        if rt.trace is not None and self.prefix:
+            rt.record(f"{self.prefix}.out", norm1.settled(stream, out))
+        return stream, out
+
+
+register_block("side_by_side_gated_stream32", SideBySideGatedStreamBlock)
 register_block("prenorm_residual", PreNormResidualBlock)
 register_block("prenorm_stream32", PreNormStreamBlock)
 register_block("outnorm_residual", OutputNormResidualBlock)

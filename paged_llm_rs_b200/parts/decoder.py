@@ -12,9 +12,10 @@ from typing import Dict, List, Optional
 
 import torch
 
-from . import (attention, block, diff_attention, embedding, feed_forward, latent_attention, mamba2, matrix_memory, norm,  # noqa: F401  (register the parts)
-               normed_attention, parallel, position, routed_feed_forward, sink_attention)
-from .base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSITION_ENCODINGS, Runtime, StepState,
+from . import (attention, block, diff_attention, embedding, feed_forward, gated_residual, latent_attention,  # noqa: F401  (register the parts)
+               linear_attention, mamba2, matrix_memory, norm, normed_attention, parallel, position, routed_feed_forward,
+               sink_attention)
+from .base import (BLOCKS, EMBEDDINGS, EXTRAS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSITION_ENCODINGS, Runtime, StepState,
                    make)
 from .spec import ModelSpec, TensorSpec
 
@@ -33,11 +34,14 @@ class DecoderModel:
             norms = {k: make(NORMS, "norm", ns, rt) for k, ns in ls.norms.items()}
             if ls.block not in BLOCKS:
                 raise KeyError(f"no block arrangement {ls.block!r} is registered; known: {sorted(BLOCKS)}")
-            self.blocks.append(BLOCKS[ls.block](mixer, ff, norms))
+            extras = {k: make(EXTRAS, "extra part", es, rt) for k, es in ls.extras.items()}
+            self.blocks.append(BLOCKS[ls.block](mixer, ff, norms, **(dict(extras=extras) if extras else {})))
             self.blocks[-1].prefix = ls.prefix
         self.final_norm = make(NORMS, "norm", spec.final_norm, rt)
         self.head = make(HEADS, "head", spec.head, rt)
+        self.pass_vectors = make(EXTRAS, "extra part", spec.pass_vectors, rt) if spec.pass_vectors is not None else None
         self.schedule = list(spec.schedule)
+        self._runs_twice = len({e.layer for e in self.schedule}) < len(self.schedule)
 
     def parts(self):
         yield from self.position_encodings.values()
@@ -47,6 +51,9 @@ class DecoderModel:
             if b.feed_forward is not None:
                 yield b.feed_forward
             yield from b.norms.values()
+            yield from b.extras.values()
+        if self.pass_vectors is not None:
+            yield self.pass_vectors
         yield self.final_norm
         yield self.head
 
@@ -56,11 +63,13 @@ class DecoderModel:
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         for p in self.parts():
             p.bind(tensors)
+        for b in self.blocks:
+            b.prepare()
 
     def cache_needs(self) -> List[Optional[object]]:
-        """Per schedule entry what its mixer needs of the cache manager; None for
+        """Per schedule entry what its block needs of the cache manager; None for
         an entry that reads another entry's cache or needs nothing."""
-        return [None if e.reads_cache_of is not None else self.blocks[e.layer].mixer.cache_need()
+        return [None if e.reads_cache_of is not None else self.blocks[e.layer].cache_need()
                 for e in self.schedule]
 
     def capturable(self) -> bool:
@@ -78,16 +87,24 @@ class DecoderModel:
         residual = self.embedding.forward(step.tokens)
         for encoding in self.position_encodings.values():
             residual = encoding.at_embedding(residual, step)
+        embedded = None
+        if any(e.add_embedding for e in self.schedule):
+            embedded = residual if all(b.keeps_stream for b in self.blocks) else residual.clone()
         delta = None
         for i, e in enumerate(self.schedule):
             own = e.reads_cache_of is None
             blk, cache = self.blocks[e.layer], caches[i if own else e.reads_cache_of]
+            if e.add_embedding or e.add_pass is not None:
+                residual, delta = blk.add_ahead(residual, delta, embedded if e.add_embedding else None,
+                                                self.pass_vectors.vector(e.add_pass) if e.add_pass is not None else None)
             if outside is not None and not getattr(blk.mixer, "graph_safe", False):
                 h = blk.pre_mixer(residual, delta)
                 a = outside(lambda blk=blk, h=h, cache=cache, own=own: blk.mixer.forward(h, step, cache, own), h)
                 residual, delta = blk.post_mixer(residual, a, step)
                 continue
             residual, delta = blk.forward(residual, delta, step, cache, own)
+            if self._runs_twice and self.rt.trace is not None and f"{blk.prefix}.out" in self.rt.trace:
+                self.rt.trace[f"run{i}.out"] = self.rt.trace[f"{blk.prefix}.out"]      # (a later run of the layer writes its name again)
         if self.schedule:
             residual, delta = self.blocks[self.schedule[-1].layer].settle(residual, delta)
         if step.n_wanted == 0:

@@ -82,6 +82,7 @@ class LinearHead(Part):
         self.tied, self.tied_to = bool(p.get("tied", False)), p.get("tied_to")
         self.leaf = p.get("leaf", "weight")
         self.scale = float(p.get("scale", 1.0))             # logits = (W x) * scale
+        self.softcap = p.get("softcap")                     # then logits = cap * tanh(logits / cap); None: not
         self.weight = None
 
     def _name(self, leaf: str) -> str:
@@ -108,6 +109,8 @@ class LinearHead(Part):
         logits = ops.linear(x, self.weight, out_dtype=torch.float32)
         if self.scale != 1.0:
             ops.scale32(logits, self.scale)
+        if self.softcap:
+            ops.softcap32(logits, float(self.softcap))
         self.rt.record(self._name("out"), logits)
         return logits
 

@@ -73,4 +73,40 @@ class SwiGLUMLP(FeedForward):
         return out
 
 
+class PolyNormMLP(FeedForward):
+    """A feed-forward without a gate, down(act(up h)) with act(u) = a N(u) + b N(u^2) + c N(u^3) + e: powers entry by entry, N
+    dividing a token's vector by its root mean square, the four numbers a tensor of the layer.  ``forward_rest`` goes on from
+    the first product's output (a column range of a wider tensor, say)."""
+
+    def __init__(self, spec, rt):
+        super().__init__(spec, rt)
+        p = spec.params
+        self.hidden, self.inter, self.eps = int(p["hidden_size"]), int(p["intermediate_size"]), float(p["eps"])
+        self.names = dict(up="up", down="down", act="act")
+        self.names.update(p.get("names", {}))
+        self.w_first = self.w_down = self.coefficients = None
+
+    def tensors(self):
+        n = self.names
+        return [TensorSpec(self._name(n["up"]), (self.inter, self.hidden)), TensorSpec(self._name(n["down"]), (self.hidden, self.inter)),
+                TensorSpec(self._name(n["act"]), (4,), "offset")]
+
+    def bind(self, tensors):
+        t = lambda k: tensors[self._name(self.names[k])]
+        self.w_first, self.w_down, self.coefficients = t("up"), t("down"), t("act")
+
+    def forward_rest(self, u, step):
+        act = torch.empty((u.shape[0], self.inter), dtype=u.dtype, device=u.device)
+        ops.poly_norm(u, self.coefficients, self.eps, act)
+        out = ops.linear(act, self.w_down, status=self.rt.status)
+        if self.rt.trace is not None:
+            for leaf, t in (("up.out", u), ("down.in", act), ("out", out)):
+                self.rt.record(self._name(leaf), t)
+        return out
+
+    def forward(self, x, step):
+        return self.forward_rest(ops.linear(x, self.w_first, status=self.rt.status), step)
+
+
 register_feed_forward("swiglu_mlp", SwiGLUMLP)
+register_feed_forward("poly_norm_mlp", PolyNormMLP)

@@ -154,7 +154,71 @@ class SandwichStreamRMSNorm(RMSNorm):
         return stream
 
 
+class PendingGated:
+    """What is still to be added to a stream whose sublayers sit side by side: the mixer's terms ((output, constant), one or
+    two) with their gate, the feed-forward's output with its gate (a gate is (logits, bias)), and what a schedule adds ahead
+    of a pass; the next norm's kernel adds it all."""
+
+    __slots__ = ("terms", "gate", "fed", "fed_gate", "embedded", "vector")
+
+    def __init__(self, terms=(), gate=None, fed=None, fed_gate=None):
+        self.terms, self.gate, self.fed, self.fed_gate = list(terms), gate, fed, fed_gate
+        self.embedded = self.vector = None
+
+    def arguments(self) -> dict:
+        a = dict(embedded=self.embedded, vector=self.vector)
+        if self.terms:
+            a.update(mixed=self.terms[0][0], mixed_scale=self.terms[0][1])
+            if len(self.terms) > 1:
+                a.update(mixed2=self.terms[1][0], mixed2_scale=self.terms[1][1])
+            if self.gate is not None:
+                a.update(mixed_gate=self.gate[0], mixed_bias=self.gate[1])
+        if self.fed is not None:
+            a.update(fed=self.fed)
+            if self.fed_gate is not None:
+                a.update(fed_gate=self.fed_gate[0], fed_bias=self.fed_gate[1])
+        return a
+
+
+class GatedStreamRMSNorm(RMSNorm):
+    """RMSNorm in a decoder whose residual stream stays float32 and whose sublayers sit side by side behind gates: its block
+    runs two of them, the token shift and the pending sum in one kernel; alone (the model's last norm) ``add_norm`` forms the
+    pending sum and norms it into the compute dtype, and ``settled`` returns the sum itself.  The stream it is given stays as
+    it is.  ``one_plus``: the file holds gain - 1.  ``optional``: the gain may be absent (a norm that nothing uses)."""
+
+    def __init__(self, spec, rt):
+        super().__init__(spec, rt)
+        self.one_plus, self.optional = bool(spec.params.get("one_plus", False)), bool(spec.params.get("optional", False))
+
+    def tensors(self):
+        return [TensorSpec(self._gain_name(), (self.width,), "gain", optional=self.optional)]
+
+    def bind(self, tensors):
+        w = tensors.get(self._gain_name())
+        self.gain = w + 1.0 if self.one_plus and w is not None else w
+
+    def forward(self, x, rows=None):
+        return self.add_norm(x, None, rows)
+
+    def add_norm(self, residual, delta, rows=None):
+        if residual.dtype != torch.float32 or not isinstance(delta, (PendingGated, type(None))):
+            raise ValueError("this norm reads a float32 stream and what its own kind of block left pending")
+        n = rows.numel() if rows is not None else residual.shape[0]
+        out = torch.empty((n, self.width), dtype=self.rt.dtype, device=residual.device)
+        ops.gated_sum_norm32(residual, self.gain, out, self.eps, rows=rows, **(delta.arguments() if delta is not None else {}))
+        self.rt.record(self._name("out"), out)
+        return out
+
+    def settled(self, stream, delta: PendingGated):
+        """The stream with all that is pending added, as a tensor of its own."""
+        x = torch.empty_like(stream)
+        ops.gated_sum_norm32(stream, self.gain, torch.empty(stream.shape, dtype=self.rt.dtype, device=stream.device), self.eps, x_out=x,
+                             **delta.arguments())
+        return x
+
+
 register_norm("rmsnorm", RMSNorm)
+register_norm("rmsnorm_gated_stream32", GatedStreamRMSNorm)
 register_norm("rmsnorm_stream32", StreamRMSNorm)
 register_norm("rmsnorm_scaled_stream32", ScaledStreamRMSNorm)
 register_norm("rmsnorm_sandwich_stream32", SandwichStreamRMSNorm)

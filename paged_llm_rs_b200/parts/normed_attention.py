@@ -12,6 +12,7 @@ With h the mixer's input, per token at position p and query head a (kv head a //
                                       the angle p * rot_base^(-2i / rot_dims); 0: no rotation
     weight(p, j) = exp(scale q . k_j) / (sink + sum over j' <= p of exp(scale q . k_j'))
                                       ``sink_one``: sink = 1 = exp(0), as if one more key scored zero and carried nothing; else 0
+                                      ``chunk``: j runs over p's own chunk of that many positions only (0: from the start)
     out = W_o ([sum over j <= p of weight(p, j) v_j]_a * sigmoid(W_g h)_a)  (``gate`` None: no such factor)
 
 A token's key and value lie side by side in one cache row (``JoinedKVNeed``); the attention itself is the kernel of the
@@ -46,6 +47,7 @@ class NormedQKAttention(Mixer):
         self.temp_coef, self.temp_every = float(p.get("temp_coef") or 0.0), int(p.get("temp_every") or 0)
         self.sink_one = bool(p.get("sink_one", False))
         self.gate = p.get("gate")
+        self.chunk = int(p.get("chunk") or 0)
         if self.qk_norm not in ops.QK_NORMS:
             raise ValueError(f"qk_norm {self.qk_norm!r}: one of {list(ops.QK_NORMS)}")
         if self.gate not in (None,) + tuple(ops.GATE_KINDS):
@@ -93,7 +95,8 @@ class NormedQKAttention(Mixer):
 
     def cache_need(self):
         if self._need is None:
-            self._need = JoinedKVNeed("full", self.nkv, self.dk, self.dv, None, 0, group_size=self.nh // self.nkv)
+            self._need = JoinedKVNeed("chunk" if self.chunk else "full", self.nkv, self.dk, self.dv, None, 0,
+                                      group_size=self.nh // self.nkv, chunk=self.chunk)
         return self._need
 
     def plan_wish(self, page_size: int):
@@ -111,7 +114,7 @@ class NormedQKAttention(Mixer):
                                self.nh, self.nkv, self.dk, self.dv, self.values_are_keys, st)
         o = torch.empty((T, self.nh * self.dv), dtype=x.dtype, device=x.device)
         ops.attention_sink(q, kv_pool, g.block_tables, g.plan, o, self.sinks, self.nh, self.nkv, self.dk, self.dv, 0, 0,
-                           self.scale, 0.0, st)
+                           self.scale, 0.0, st, chunk=self.chunk)
         if self.gate:
             ops.gate_mul(o, proj[:, self.g_off:self.g_off + self.nh * self.dv], self.gate)
         out = ops.linear(o, self.w_o, status=st)

@@ -44,6 +44,11 @@ class ParallelMixers(Mixer):
     def cache_need(self):
         return CompositeNeed(tuple(p.cache_need() for p in self.parts))
 
+    def forward_terms(self, x, step, cache, writes_cache=True):
+        """[(output, constant)] for a block whose next kernel forms the sum; two parts at most."""
+        terms = [(p.forward(x, step, c, writes_cache), s) for p, c, s in zip(self.parts, cache, self.scales)]
+        return terms if len(terms) == 2 else [(self.forward(x, step, cache, writes_cache), 1.0)]
+
     def forward(self, x, step, cache, writes_cache=True):
         outs = [p.forward(x, step, c, writes_cache) for p, c in zip(self.parts, cache)]
         acc = ops.scaled_sum2(outs[0], outs[1], self.scales[0], self.scales[1])

@@ -28,18 +28,18 @@ def check_tensors(specs: Iterable[TensorSpec], available: Dict[str, tuple]) -> N
     specs = list(specs)
     wanted = {}
     for s in specs:
-        if s.name in wanted and wanted[s.name].shape != tuple(s.shape):
+        if s.name in wanted and tuple(wanted[s.name].shape) != tuple(s.shape):
             raise WeightError(f"two parts ask for {s.name} at different shapes")
         # a tensor is optional only if every part asking for it says so
         if s.name in wanted:
-            s = TensorSpec(s.name, tuple(s.shape), s.role, s.optional and wanted[s.name].optional)
+            s = TensorSpec(s.name, tuple(s.shape), s.role, s.optional and wanted[s.name].optional, s.drawn)
         wanted[s.name] = s
     missing = [n for n, s in wanted.items() if n not in available and not s.optional]
     unexpected = [n for n in available if n not in wanted]
     wrong = [
         f"{n} has shape {list(available[n])}, expected {list(s.shape)}"
         for n, s in wanted.items()
-        if n in available and tuple(available[n]) != tuple(s.shape)
+        if n in available and not s.fits(tuple(available[n]))
     ]
     if missing or unexpected or wrong:
         lines = ["the weight file does not fit the model:"]

@@ -60,14 +60,15 @@ def random_tensors(model_spec, seed: int, dtype: torch.dtype = torch.bfloat16, d
     for s in tensor_specs_of(model_spec):
         if s.name in out or (s.optional and not write_optional):
             continue
+        shape = s.drawn or s.shape
         if s.role == "gain":
-            t = 1.0 + gain_std * _standard_normal(seed, s.name, s.shape, device)
+            t = 1.0 + gain_std * _standard_normal(seed, s.name, shape, device)
         elif s.role == "offset":
-            t = gain_std * _standard_normal(seed, s.name, s.shape, device)
+            t = gain_std * _standard_normal(seed, s.name, shape, device)
         elif s.role == "index":
-            t = torch.zeros(s.shape, dtype=torch.int32, device=device)
+            t = torch.zeros(shape, dtype=torch.int32, device=device)
         else:
-            t = matrix_std * _standard_normal(seed, s.name, s.shape, device)
+            t = matrix_std * _standard_normal(seed, s.name, shape, device)
         out[s.name] = t if s.role == "index" else t.to(dtype)
     return out
 
