@@ -186,7 +186,7 @@ class MixerRig:
         bound = {}
         for s in self.mixer.tensors():
             t = tensors[s.name]
-            assert tuple(t.shape) == tuple(s.shape), s.name
+            assert s.fits(tuple(t.shape)), s.name
             bound[s.name] = (t.to(dtype) if s.role == "matrix" else t.float()).to(DEV)
         self.mixer.bind(bound)
         self.cache = CacheManager([self.mixer.cache_need()], page, pages, max_requests, dtype, DEV, prefix_cache=False)
