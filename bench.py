@@ -1181,6 +1181,202 @@ def tebozen_kernels(z, pk):
     return out
 
 
+# ---- the retention / chunked-attention-beside-gated-linear-attention decoder (Reperax) ----------------------------------
+# Sizes that resemble real layers, at the widths of the 0.6B and of a 2B-class shape: retention of width / 256 heads with
+# keys of 128 (all rotated) and values of 256 entries; chunked attention of sixteen heads over eight kv heads of 128 with
+# values of 64, in chunks of 1024, beside gated linear attention of width / 128 heads of 128 x 128 with a decay of inner
+# size 16; a feed-forward without a gate.  Layers alternate and are run once, ahead of them the pass's vector.  The other
+# model is Pamarax at the same width, depth, head sizes, feed-forward and vocabulary, its matrix LSTM layers in the place of
+# retention, its side-by-side layers (attention over the whole context, gated delta rule) in the place of the side-by-side ones.
+REPERAX_SIZES = {
+    "1024": dict(width=1024, heads=16, kv_heads=8, dim=128, vdim=64, chunk=1024, r_heads=4, r_dim=128, r_vdim=256, g_heads=8, g_dim=128,
+                 g_vdim=128, rank=16, ff=3072),
+    "2048": dict(width=2048, heads=16, kv_heads=8, dim=128, vdim=64, chunk=1024, r_heads=8, r_dim=128, r_vdim=256, g_heads=16, g_dim=128,
+                 g_vdim=128, rank=16, ff=6144),
+}
+
+
+def reperax_config(z, layers):
+    ret = dict(heads=z["r_heads"], dim=z["r_dim"], vdim=z["r_vdim"], rot=dict(dims=z["r_dim"], base=10000.0),
+               decay=[1.0 - 2.0 ** -(5 + i * 5 / max(1, z["r_heads"] - 1)) for i in range(z["r_heads"])])
+    left = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["vdim"], scale=z["dim"] ** -0.5, mask=dict(size=z["chunk"]))
+    right = dict(heads=z["g_heads"], dim=z["g_dim"], vdim=z["g_vdim"], tau=16.0)
+    cycle = [dict(type="retention", mixer=ret), dict(type="parallel", mixer=dict(left=left, right=right, left_scale=0.8, right_scale=0.6))]
+    return dict(architecture="Reperax", vocab=LATENT_VOCAB, width=z["width"], norm=dict(eps=1e-6), logit_softcap=30.0,
+                loop=dict(start=0, stop=layers, times=1), layers=[dict(cycle[i % 2], mlp=dict(kind="dense", ff=z["ff"])) for i in range(layers)])
+
+
+def reperax_beside_matrix(size, layers, pk, clocks, steps, warmup, which="both"):
+    """Decode (batch 1, 8, 64 at context 4096) and the 2048-token prefill of the Reperax shape ``size`` and of the Pamarax shape
+    of the same width, layers, head sizes, feed-forward and vocabulary: tokens a second, side by side; then Reperax's own
+    kernels alone beside the like kernels of Pamarax."""
+    import gc
+    import torch
+    from paged_llm_rs_b200 import Engine, write_random_model
+
+    z = REPERAX_SIZES[size]
+    mz = MATRIX_SIZES[size]
+    matrix = matrix_config(mz, 4)
+    matrix["layers"] = [matrix["layers"][1 + i % 2] for i in range(layers)]        # matrix LSTM, side by side, ...
+    out = dict(size=size, layers=layers, vocab=LATENT_VOCAB, reperax=dict(z))
+    for name, cfg in (("reperax", reperax_config(z, layers)), ("pamarax", matrix)):
+        if which not in ("both", name):
+            continue
+        tmp = tempfile.mkdtemp(prefix="pllm_bench_", dir=scratch_dir())
+        try:
+            model_dir = write_random_model(os.path.join(tmp, "model"), cfg, 0, device="cuda")
+            ctx = 4096
+            pages = 64 * (ctx // PAGE + 4) + (PREFILL_TOKENS + 1024) // PAGE + 64
+            eng = Engine(model_dir, dtype="bfloat16", block_size=PAGE, blocks=pages, max_batch=64, chunk=PREFILL_TOKENS,
+                         prefix_cache=False)
+            shutil.rmtree(tmp, ignore_errors=True)
+            runner = eng.runner
+            for g in runner.cache.groups:
+                if g.pool is not None:
+                    g.pool.normal_(0.0, 1.0)
+            res = dict(weight_bytes=runner.weight_bytes(), cache_bytes_a_token=runner.cache.bytes_per_token())
+            for b in (1, 8, 64):
+                ms, launches, spread = decode_point(runner, b, ctx, max(5, steps // 2), warmup, clocks, repeats=4)
+                res[f"decode_b{b}_tok_s"] = round(b / (spread["median_ms"] / 1e3), 1)
+                res[f"decode_b{b}_ms"] = spread["median_ms"]
+                res[f"decode_b{b}_launches"] = launches
+            pms, _ = prefill_point(runner, LATENT_VOCAB, clocks, repeats=4)
+            res["prefill_ms"] = round(pms, 3)
+            res["prefill_tok_s"] = round(PREFILL_TOKENS / (pms / 1e3), 1)
+            out[name] = res
+            del eng, runner
+        finally:
+            shutil.rmtree(tmp, ignore_errors=True)
+            gc.collect()
+            torch.cuda.empty_cache()
+    out["kernels"] = reperax_kernels(z, pk)
+    like = matrix_kernels(mz, pk)
+    out["kernels"].update({f"pamarax_{k}": v for k, v in like.items()})
+    return out
+
+
+def reperax_kernels(z, pk):
+    """Reperax's own kernels alone, at the sizes of ``z``, each beside its like kernel of another design where that is not among
+    Pamarax's: device time (CUDA events, the median of nine after three warm-ups, an L2 flush before each), the algorithmic
+    bytes and FLOPs, and the fraction of the measured copy bandwidth or bfloat16 product rate they come to."""
+    import numpy as np
+    import torch
+    from paged_llm_rs_b200.kernels import attention_plan, ops
+    from paged_llm_rs_b200.parts.base import AttentionWork
+
+    dev, bf = "cuda", torch.bfloat16
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    target = 2 * ops.sm_count()
+    out = {}
+
+    def timed(fn):
+        for _ in range(3):
+            fn()
+        torch.cuda.synchronize()
+        ts = []
+        for _ in range(9):
+            flush_l2()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record(); fn(); b.record()
+            torch.cuda.synchronize()
+            ts.append(a.elapsed_time(b))
+        return statistics.median(ts)
+
+    def note(name, ms, nbytes, flops):
+        r = dict(us=round(ms * 1e3, 2), mbytes=round(nbytes / 1e6, 2), gflop=round(flops / 1e9, 3),
+                 hbm_frac=round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 4),
+                 bf16_frac=round(flops / (ms / 1e3) / 1e12 / pk["bf16_tflops"], 4))
+        r["frac_of_slower_bound"] = round(max(r["hbm_frac"], r["bf16_frac"]), 4)
+        out[name] = r
+
+    def plan(segs, tile, ctas, window=0, chunk=0):
+        work, red, parts = attention_plan.plan_attention(segs, tile, window, ctas, target, chunk=chunk)
+        wd = torch.from_numpy(np.ascontiguousarray(work)).reshape(-1, 8).to(dev)
+        rd = torch.from_numpy(np.ascontiguousarray(red)).reshape(-1, 4).to(dev) if len(red) else torch.zeros(1, 4, dtype=torch.int32, device=dev)
+        singles = all(n == 1 for _, n, _ in segs)
+        return lambda heads, hd: AttentionWork(wd, torch.tensor([len(work)], dtype=torch.int32, device=dev), len(work), rd,
+                                                torch.tensor([len(red)], dtype=torch.int32, device=dev), len(red),
+                                                torch.zeros(max(parts, 1), heads, hd, device=dev), torch.zeros(max(parts, 1), heads, 2, device=dev),
+                                                kinds=1 if singles else 2, many_splits=attention_plan.many_splits(len(segs), ctas, target))
+
+    ctx, B, T, W = 4096, 64, PREFILL_TOKENS, z["width"]
+    n_pages = B * ctx // PAGE
+    tables = torch.randperm(n_pages, dtype=torch.int32).view(B, ctx // PAGE).to(dev)
+    cases = {"decode_b64_ctx4096": [(i, 1, ctx - 1) for i in range(B)], "prefill_2048": [(0, T, 0)]}
+    # -- attention in chunks, beside the same kernel with a window of the chunk's size
+    nh, nkv, dk, dv, chunk = z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["chunk"]
+    pool = torch.randn(n_pages, nkv, PAGE, dk + dv, device=dev).to(bf)
+    tile, ctas = ops.attention_sink_tile_tokens(nh, nkv, bf, dk, dv), ops.attention_sink_ctas_per_item(nh, nkv, bf, dk, dv)
+    for case, segs in cases.items():
+        n = sum(c for _, c, _ in segs)
+        q, o = torch.randn(n, nh * dk, device=dev).to(bf), torch.empty(n, nh * dv, dtype=bf, device=dev)
+        for label, win, ch in (("attention_chunked", 0, chunk), ("like_attention_window", chunk, 0)):
+            seen = lambda p: p % chunk + 1 if ch else min(p + 1, chunk)
+            keys = sum(seen(p + i) for _, c, p in segs for i in range(c))
+            seg_keys = sum((p + c) - (p - p % chunk if ch else max(0, p - chunk + 1)) for _, c, p in segs)
+            w = plan(segs, tile, ctas, win, ch)(nh, dv)
+            ms = timed(lambda: ops.attention_sink(q, pool, tables, w, o, None, nh, nkv, dk, dv, win, 0, dk ** -0.5, 0.0, status, chunk=ch))
+            note(f"{label}_{case}", ms, seg_keys * nkv * (dk + dv) * 2 + n * nh * (dk + dv) * 2, 2 * nh * (dk + dv) * keys)
+        # q/k norm over the projection and the cache write
+        k_off, v_off = nh * dk, (nh + nkv) * dk
+        proj = torch.randn(n, v_off + nkv * dv, device=dev).to(bf)
+        gq, gk = torch.ones(nh * dk, device=dev), torch.ones(nkv * dk, device=dev)
+        pos = torch.arange(n, dtype=torch.int32, device=dev)
+        slots = torch.randperm(n_pages * PAGE, dtype=torch.int32)[:n].to(dev)
+        ms = timed(lambda: ops.normed_qk_kv_write(proj, k_off, v_off, q, gq, gk, "projection", 1e-6, 0.0, 0, None, 0, pos, slots, pool,
+                                                  nh, nkv, dk, dv, False, status))
+        note(f"normed_qk_kv_write_{case}", ms, 2 * proj.numel() * 2, 0)
+    del pool
+    # -- the recurrences between their projections
+    for label, H, d, E, channel in (("retention", z["r_heads"], z["r_dim"], z["r_vdim"], False), ("gated_linear", z["g_heads"], z["g_dim"], z["g_vdim"], True)):
+        floats = ops.linear_attention_state_floats(H, d, E)
+        state = torch.zeros(B + 1, floats, device=dev)
+        inv = torch.rand(d // 2, device=dev)
+        decay = torch.full((H,), 0.99, device=dev)
+        a2, ab, gain = torch.randn(H * d, z["rank"], device=dev).to(bf), torch.full((H * d,), 3.0, device=dev), torch.ones(E, device=dev)
+        for case, segs in cases.items():
+            n = sum(c for _, c, _ in segs)
+            u = torch.randn(n, 2 * H * d + 2 * H * E, device=dev).to(bf)
+            a1 = torch.randn(n, z["rank"], device=dev)
+            sg = torch.tensor([(t0, c, p, i + 1) for i, (t0, c, p) in enumerate(segs)], dtype=torch.int32, device=dev)
+            y = torch.empty(n, H * E, dtype=bf, device=dev)
+            longest = max(c for _, c, _ in segs)
+            args = (u, 0, H * d, 2 * H * d, 2 * H * d + H * E)
+            if channel:
+                run = lambda: ops.linear_attention_mix(*args, d ** -0.5, 1.0, 0, None, None, a1, a2, ab, 16.0, gain, sg, longest, state, y, H, d, E, 1e-6)
+            else:
+                run = lambda: ops.linear_attention_mix(*args, 1.0, d ** -0.5, d, inv, decay, None, None, None, 1.0, None, sg, longest, state, y, H, d, E, 1e-6)
+            ms = timed(run)
+            # (counted as for the like recurrences: the read-out in float written and read once, the state read and written)
+            note(f"{label}_mix_{case}", ms, u.numel() * 2 + (a1.numel() * 4 if channel else 0) + n * H * E * 4 * 2 + y.numel() * 2 + len(segs) * floats * 4 * 2,
+                 6 * n * H * d * E)
+        del state
+    # -- the gated sum, two norms and the shift; the polynomial activation beside silu(gate + b) * (up + b); the logits' cap
+    ff = z["ff"]
+    for case, n in (("decode_b64", B), ("prefill_2048", T)):
+        x, xo = torch.randn(n, W, device=dev), torch.empty(n, W, device=dev)
+        new = lambda: torch.randn(n, W, device=dev).to(bf)
+        a1, a2, f, gate, y1, ys, y2 = new(), new(), new(), new(), new(), new(), new()
+        wide = torch.randn(n, ff + W, device=dev).to(bf)
+        vec = torch.ones(W, device=dev)
+        sg = torch.tensor([(i, 1, 9, i + 1) for i in range(B)] if n == B else [(0, n, 0, 1)], dtype=torch.int32, device=dev)
+        st = torch.zeros(B + 1, W, device=dev)
+        ms = timed(lambda: ops.gated_sum_norm32(x, vec, y1, 1e-6, mixed=a1, mixed_scale=0.8, mixed2=a2, mixed2_scale=0.6, mixed_gate=gate, mixed_bias=vec,
+                                                fed=f, fed_gate=wide[:, ff:], fed_bias=vec, x_out=xo, shift=vec, shifted=ys, segments=sg, state=st,
+                                                gain2=vec, out2=y2))
+        note(f"gated_sum_norm32_{case}", ms, n * W * (4 + 4 + 5 * 2 + 3 * 2) + sg.shape[0] * W * 8, 0)
+        act = torch.empty(n, ff, dtype=bf, device=dev)
+        ms = timed(lambda: ops.poly_norm(wide[:, :ff], vec[:4].contiguous(), 1e-6, act))
+        note(f"poly_norm_{case}", ms, 2 * n * ff * 2, 0)
+        gu, bias = torch.randn(n, 2 * ff, device=dev).to(bf), torch.zeros(2 * ff, device=dev)
+        ms = timed(lambda: ops.swiglu_bias(gu, bias, act))
+        note(f"like_swiglu_bias_{case}", ms, 3 * n * ff * 2, 0)
+    logits = torch.randn(B, LATENT_VOCAB, device=dev)
+    note("softcap32_decode_b64", timed(lambda: ops.softcap32(logits, 30.0)), logits.numel() * 8, 0)
+    note("like_scale32_decode_b64", timed(lambda: ops.scale32(logits, 1.0)), logits.numel() * 8, 0)
+    return out
+
+
 TRACE_KERNELS = {0: "(tcgen05 kernel)", 1: "embed", 2: "rmsnorm", 3: "swiglu", 4: "qk_norm_rope_kv", 5: "attention_generic", 6: "attention_reduce",
                  7: "attention_mma", 8: "attention_tma", 9: "skinny_gemm", 10: "sample_partial", 11: "sample_final", 12: "gemm_tcgen05", 13: "attention_tcgen05"}
 TRACE_FILES = ["elementwise", "qk_norm_rope_kv", "attention_generic", "attention_mma", "attention_decode_tma", "sampling",
@@ -1344,8 +1540,11 @@ def main(argv=None) -> int:
     ap.add_argument("--tebozen-size", choices=sorted(TEBOZEN_SIZES), default="1024",
                     help="with --only tebozen: the width of the differential-attention / matrix-LSTM / latent-attention decoder (Tebozen)")
     ap.add_argument("--tebozen-model", choices=["both", "tebozen", "bumisun"], default="both", help="with --only tebozen: one model alone")
+    ap.add_argument("--reperax-size", choices=sorted(REPERAX_SIZES), default="1024",
+                    help="with --only reperax: the width of the retention / chunked-attention-beside-gated-linear-attention decoder (Reperax)")
+    ap.add_argument("--reperax-model", choices=["both", "reperax", "pamarax"], default="both", help="with --only reperax: one model alone")
     ap.add_argument("--only", choices=["decode", "prefill", "long-prompt", "timeline", "reference-kernel", "plain-cpu", "latent", "hybrid", "matrix",
-                                       "tebozen"],
+                                       "tebozen", "reperax"],
                     default=None,
                     help="run one part alone and print a short line (for profiling; not a bench record); "
                          "long-prompt: a prompt of --context tokens in portions of 2048, each portion timed; "
@@ -1359,7 +1558,9 @@ def main(argv=None) -> int:
                          "(Pamarax: gated attention, matrix LSTM, attention beside a gated delta rule) beside the Bumisun shape of "
                          "equal size, with its own kernels timed alone beside Bumisun's like ones (--matrix-size, --layers, default 8); "
                          "tebozen: the same for the decoder of differential attention, matrix LSTM and latent attention layers with "
-                         "squared-relu experts (Tebozen) beside the Bumisun shape of equal size (--tebozen-size, --layers, default 8)")
+                         "squared-relu experts (Tebozen) beside the Bumisun shape of equal size (--tebozen-size, --layers, default 8); "
+                         "reperax: the same for the decoder of retention layers and chunked attention beside gated linear attention "
+                         "(Reperax) beside the Pamarax shape of equal size (--reperax-size, --layers, default 8)")
     args = ap.parse_args(argv)
 
     if args.impl == "reference":
@@ -1407,6 +1608,12 @@ def main(argv=None) -> int:
     if args.only == "tebozen":
         clocks.start()
         out = tebozen_beside_hybrid(args.tebozen_size, args.layers or 8, pk, clocks, steps, warmup, which=args.tebozen_model)
+        out["clocks"] = clocks.stop()
+        print(json.dumps(out))
+        return 0
+    if args.only == "reperax":
+        clocks.start()
+        out = reperax_beside_matrix(args.reperax_size, args.layers or 8, pk, clocks, steps, warmup, which=args.reperax_model)
         out["clocks"] = clocks.stop()
         print(json.dumps(out))
         return 0
