@@ -1342,10 +1342,11 @@ def reperax_kernels(z, pk):
             y = torch.empty(n, H * E, dtype=bf, device=dev)
             longest = max(c for _, c, _ in segs)
             args = (u, 0, H * d, 2 * H * d, 2 * H * d + H * E)
+            rope = ops.rope_table(torch.arange(n, dtype=torch.int32, device=dev), inv)          # (once a step, for all layers)
             if channel:
                 run = lambda: ops.linear_attention_mix(*args, d ** -0.5, 1.0, 0, None, None, a1, a2, ab, 16.0, gain, sg, longest, state, y, H, d, E, 1e-6)
             else:
-                run = lambda: ops.linear_attention_mix(*args, 1.0, d ** -0.5, d, inv, decay, None, None, None, 1.0, None, sg, longest, state, y, H, d, E, 1e-6)
+                run = lambda: ops.linear_attention_mix(*args, 1.0, d ** -0.5, d, inv, decay, None, None, None, 1.0, None, sg, longest, state, y, H, d, E, 1e-6, rope=rope)
             ms = timed(run)
             # (counted as for the like recurrences: the read-out in float written and read once, the state read and written)
             note(f"{label}_mix_{case}", ms, u.numel() * 2 + (a1.numel() * 4 if channel else 0) + n * H * E * 4 * 2 + y.numel() * 2 + len(segs) * floats * 4 * 2,

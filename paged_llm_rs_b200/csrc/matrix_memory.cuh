@@ -32,7 +32,23 @@ __device__ __forceinline__ void mm_fetch16(const bf16* p, float* dst, float scal
 // A warp a (token, head): o / rms(o) * gain * act(gate).  y float [tokens, H e]; gate: [tokens, g_stride] of the compute dtype;
 // gain_per_head: the gain has H e entries, else e entries shared by the heads (null: no gain); kind 0 sigmoid, 1 silu.  With dn ([tokens, H, 2]:
 // the normaliser's product with the query, exp(-m)) y holds numerators, and o = y / (max(|n . q|, exp(-m)) + 1e-6).
-template <typename T>
+// N: entries a lane takes at a time (4 where rows are whole vectors of four, else 1).
+__device__ __forceinline__ void head_quad_load(const float* p, float* v) {
+    const float4 r = *reinterpret_cast<const float4*>(p);
+    v[0] = r.x; v[1] = r.y; v[2] = r.z; v[3] = r.w;
+}
+__device__ __forceinline__ void head_quad_load(const bf16* p, float* v) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(r.x << 16); v[1] = __uint_as_float(r.x & 0xffff0000u);
+    v[2] = __uint_as_float(r.y << 16); v[3] = __uint_as_float(r.y & 0xffff0000u);
+}
+__device__ __forceinline__ void head_quad_store(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void head_quad_store(bf16* p, const float* v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+template <typename T, int N>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* y, const float* __restrict__ dn, const T* gate, int g_stride,
                                                              const float* __restrict__ gain, T* __restrict__ out, long long n_rows,
                                                              int H, int E, int gain_per_head, int kind, float eps) {
@@ -45,15 +61,49 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* y, con
     const int h = (int)(r % H);
     const float* yr = y + r * E;
     const T* gr = gate + t * g_stride + (size_t)h * E;
+    const float* gn = gain ? gain + (gain_per_head ? (size_t)h * E : 0) : nullptr;
     const float over = dn ? fmaxf(fabsf(dn[r * 2]), dn[r * 2 + 1]) + 1e-6f : 1.0f;
+    constexpr int KEEP = N == 4 ? 4 : 8;          // rounds of a row that stay in registers
+    float keep[KEEP][N];
     float ss = 0.f;
-    for (int i = lane; i < E; i += 32) { const float v = yr[i] / over; ss += v * v; }
+#pragma unroll
+    for (int j = 0; j < KEEP; j++) {
+        const int i = (lane + 32 * j) * N;
+        if (i >= E) break;
+        if constexpr (N == 4) head_quad_load(yr + i, keep[j]); else keep[j][0] = yr[i];
+#pragma unroll
+        for (int k = 0; k < N; k++) { keep[j][k] /= over; ss += keep[j][k] * keep[j][k]; }
+    }
+    for (int i = (lane + 32 * KEEP) * N; i < E; i += 32 * N)
+        for (int k = 0; k < N; k++) { const float v = yr[i + k] / over; ss += v * v; }
     ss = warp_sum(ss);
     const float inv = 1.0f / sqrtf(ss / (float)E + eps);
-    for (int i = lane; i < E; i += 32) {
-        const float z = to_f32(gr[i]);
-        const float sg = mm_sigmoid(z);
-        out[r * E + i] = from_f32<T>(yr[i] / over * inv * (gain ? gain[gain_per_head ? h * E + i : i] : 1.0f) * (kind == 1 ? z * sg : sg));
+    auto finish = [&](int i, float* v) {
+        float z[N], g[N];
+        if constexpr (N == 4) {
+            head_quad_load(gr + i, z);
+            if (gn) head_quad_load(gn + i, g);
+        } else {
+            z[0] = to_f32(gr[i]);
+            if (gn) g[0] = gn[i];
+        }
+#pragma unroll
+        for (int k = 0; k < N; k++) {
+            const float sg = mm_sigmoid(z[k]);
+            v[k] = v[k] * inv * (gn ? g[k] : 1.0f) * (kind == 1 ? z[k] * sg : sg);
+        }
+        if constexpr (N == 4) head_quad_store(out + r * E + i, v); else out[r * E + i] = from_f32<T>(v[0]);
+    };
+#pragma unroll
+    for (int j = 0; j < KEEP; j++) {
+        const int i = (lane + 32 * j) * N;
+        if (i >= E) break;
+        finish(i, keep[j]);
+    }
+    for (int i = (lane + 32 * KEEP) * N; i < E; i += 32 * N) {
+        float v[N];
+        for (int k = 0; k < N; k++) v[k] = yr[i + k] / over;
+        finish(i, v);
     }
 }
 
@@ -61,7 +111,13 @@ template <typename T>
 static void launch_head_norm_gate(const float* y, const float* dn, const void* gate, int g_stride, const float* gain, void* out, int n_tokens, int H, int E,
                                   int gain_per_head, int kind, float eps, cudaStream_t stream) {
     const long long rows = (long long)n_tokens * H;
-    launch_chained(head_norm_gate_kernel<T>, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, stream, y, dn, (const T*)gate, g_stride, gain,
-                   (T*)out, rows, H, E, gain_per_head, kind, eps);
+    const bool quads = E % 4 == 0 && g_stride % 4 == 0 && (((uintptr_t)y | (uintptr_t)gain | (uintptr_t)out) & 15) == 0 &&
+                       ((uintptr_t)gate & (4 * sizeof(T) - 1)) == 0;
+    const dim3 grid((unsigned)((rows + 7) / 8));
+    if (quads)
+        launch_chained(head_norm_gate_kernel<T, 4>, grid, dim3(256), 0, stream, y, dn, (const T*)gate, g_stride, gain, (T*)out, rows, H, E,
+                       gain_per_head, kind, eps);
+    else
+        launch_chained(head_norm_gate_kernel<T, 1>, grid, dim3(256), 0, stream, y, dn, (const T*)gate, g_stride, gain, (T*)out, rows, H, E,
+                       gain_per_head, kind, eps);
 }
-

@@ -115,7 +115,8 @@ def lib():
                                         c_int, P, c_ll, P, c_int, c_int, c_float, P]
         sig["pllm_poly_norm"] = [c_int, P, c_int, P, P, c_int, c_int, c_float, P]
         sig["pllm_softcap32"] = [P, c_float, c_ll, P]
-        sig["pllm_linear_attention_mix"] = [c_int, P] + [c_int] * 5 + [c_float, c_float, c_int, P, P, P, P, P, c_int, c_float, P, P, c_int, c_int, P, c_ll,
+        sig["pllm_rope_table"] = [P, P, P, c_int, c_int, P]
+        sig["pllm_linear_attention_mix"] = [c_int, P] + [c_int] * 5 + [c_float, c_float, c_int, P, P, P, P, P, P, c_int, c_float, P, P, c_int, c_int, P, c_ll,
                                             P, P, P] + [c_int] * 4 + [c_float, P]
         wide = {"pllm_linear_attention_state_floats": [c_int] * 3, "pllm_linear_attention_scratch_floats": [c_int] * 6,
                 "pllm_mlstm_state_floats": [c_int] * 3, "pllm_delta_state_floats": [c_int] * 5}
@@ -1535,18 +1536,29 @@ def linear_attention_state_floats(heads: int, dim: int, vdim: int) -> int:
     return heads * dim * vdim
 
 
+def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
+    """cos and sin of position * inv_freq[i] (a float32 product) for every token: float32 [T, len(inv_freq), 2]."""
+    _dev(positions, inv_freq)
+    _i32(positions, "positions"); _f32(inv_freq, "inv_freq")
+    T, half = positions.numel(), inv_freq.numel()
+    out = torch.empty((T, half, 2), dtype=torch.float32, device=positions.device)
+    _check(lib().pllm_rope_table(_ptr(positions), _ptr(inv_freq), _ptr(out), T, half, _stream()), "rope_table")
+    return out
+
+
 def linear_attention_mix(u: torch.Tensor, q_off: int, k_off: int, v_off: int, gate_off: int, q_scale: float, k_scale: float, rot: int,
                          inv_freq: Optional[torch.Tensor], decay: Optional[torch.Tensor], a1: Optional[torch.Tensor],
                          a2: Optional[torch.Tensor], a_bias: Optional[torch.Tensor], tau: float, gain: Optional[torch.Tensor],
                          segments: torch.Tensor, max_segment_tokens: int, state: torch.Tensor, out: torch.Tensor, heads: int, dim: int,
-                         vdim: int, eps: float) -> torch.Tensor:
+                         vdim: int, eps: float, rope: Optional[torch.Tensor] = None) -> torch.Tensor:
     """From a stacked projection ``u`` [T, width] (q and k [heads dim], v and the gate [heads vdim] at the given columns) to the
     output projection's input [T, heads vdim]: q and k times their scales, turned on their first ``rot`` entries; per head
     S <- diag(alpha) S + k v^T, o = S^T q over each segment's tokens from and into its state slot; each head over its root mean
     square, the gain (vdim entries shared by the heads, or None), silu(gate).  alpha: ``decay`` (float32 [heads]), or, where
     that is None, sigmoid(a2 a1 + a_bias)^(1 / tau) a key entry with a1 float32 [T, rank] and a2 [heads dim, rank].
-    ``max_segment_tokens`` bounds a segment's tokens (1: the form for decoded tokens)."""
-    _dev(u, inv_freq, decay, a1, a2, a_bias, gain, segments, state, out)
+    ``max_segment_tokens`` bounds a segment's tokens (1: the form for decoded tokens, which forms its angles from inv_freq; the
+    other one reads them from ``rope``, the step's ``rope_table``)."""
+    _dev(u, inv_freq, rope, decay, a1, a2, a_bias, gain, segments, state, out)
     for t, n in ((inv_freq, "inv_freq"), (decay, "decay"), (a1, "a1"), (a_bias, "a_bias"), (gain, "gain"), (state, "state")):
         _f32(t, n)
     _segments_ok(segments, "linear_attention_mix")
@@ -1557,6 +1569,8 @@ def linear_attention_mix(u: torch.Tensor, q_off: int, k_off: int, v_off: int, ga
         raise KernelError("linear_attention_mix: out must be [T, heads vdim] of u's dtype")
     if rot and (inv_freq is None or inv_freq.numel() * 2 != rot):
         raise KernelError("linear_attention_mix: inv_freq must hold rot / 2 frequencies")
+    if rot and int(max_segment_tokens) != 1 and (rope is None or rope.shape != (T, rot // 2, 2) or rope.dtype != torch.float32):
+        raise KernelError("linear_attention_mix: portions of prompts need the step's rope_table, [T, rot / 2, 2] float32")
     rank = 0
     if decay is not None:
         if decay.numel() != heads:
@@ -1582,7 +1596,7 @@ def linear_attention_mix(u: torch.Tensor, q_off: int, k_off: int, v_off: int, ga
         launches = 2 + (decay is None) + (2 if floats > alpha_only else 0)
     _check(lib().pllm_linear_attention_mix(
         _code(u), _ptr(u), width, int(q_off), int(k_off), int(v_off), int(gate_off), float(q_scale), float(k_scale), int(rot), _ptr(inv_freq),
-        _ptr(decay), _ptr(a1), _ptr(a2), _ptr(a_bias), rank, 1.0 / float(tau) if decay is None else 1.0, _ptr(gain), _ptr(segments),
+        _ptr(rope), _ptr(decay), _ptr(a1), _ptr(a2), _ptr(a_bias), rank, 1.0 / float(tau) if decay is None else 1.0, _ptr(gain), _ptr(segments),
         segments.shape[0], longest, _ptr(state), state.stride(0), _ptr(scratch), _ptr(y_buf), _ptr(out), T, heads, dim, vdim, float(eps),
         _stream()), "linear_attention_mix", launches=launches)
     return out

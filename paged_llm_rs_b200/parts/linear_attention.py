@@ -67,11 +67,17 @@ class LinearAttention(Mixer):
         st = self.rt.status
         u = ops.linear(x, self.w_in, status=st)
         a1 = ops.linear(x, self.w_a1, out_dtype=torch.float32, status=st) if self.decay is None else None
+        rope = None
+        if self.rot and step.max_segment_tokens != 1:       # one table a step for all layers that turn alike
+            key = f"rope_table/{self.rot}/{self.rot_base}"
+            rope = step.carry.get(key)
+            if rope is None:
+                rope = step.carry[key] = ops.rope_table(step.positions[:x.shape[0]], self.inv_freq)
         y = torch.empty((x.shape[0], self.heads * self.vdim), dtype=x.dtype, device=x.device)
         ops.linear_attention_mix(u, **self.offsets, q_scale=self.q_scale, k_scale=self.k_scale, rot=self.rot, inv_freq=self.inv_freq,
                                  decay=self.decay, a1=a1, a2=self.w_a2, a_bias=self.a_bias, tau=self.tau, gain=self.gain,
                                  segments=step.segments, max_segment_tokens=step.max_segment_tokens, state=cache, out=y,
-                                 heads=self.heads, dim=self.dim, vdim=self.vdim, eps=self.eps)
+                                 heads=self.heads, dim=self.dim, vdim=self.vdim, eps=self.eps, rope=rope)
         out = ops.linear(y, self.w_o, status=st)
         if self.rt.trace is not None:
             for leaf, t in (("in.out", u), ("o.in", y), ("out", out)):

@@ -139,11 +139,15 @@ def kernel_recurrence(dtype, H, d, e, cuts, pad, rot, channel, seed, decay=None,
     inv = torch.tensor([base ** (-2.0 * i / rot) for i in range(rot // 2)], dtype=torch.float64).float() if rot else None
     slots = torch.randn(len(cuts) + 2, H * d * e, generator=g) if state is None else state
     st, out = slots.clone().to(DEV), torch.empty(T, H * e, dtype=dtype, device=DEV)
-    qs, ks = (d ** -0.5, 1.0) if channel else (1.0, d ** -0.5)
     dv = lambda t: None if t is None else t.to(DEV)
+    qs, ks = (d ** -0.5, 1.0) if channel else (1.0, d ** -0.5)
+    positions = torch.zeros(T, dtype=torch.int32)
+    for t0, n, before, _ in segs.tolist():
+        positions[t0:t0 + n] = torch.arange(before, before + n, dtype=torch.int32)
+    rope = ops.rope_table(positions.to(DEV), dv(inv)) if rot else None
     ops.linear_attention_mix(u.to(DEV), 0, H * d, 2 * H * d, 2 * H * d + H * e, qs, ks, rot, dv(inv), None if channel else torch.tensor(decay, device=DEV),
                              dv(a1) if channel else None, dv(a2) if channel else None, dv(ab) if channel else None, tau, dv(gain), segs.to(DEV),
-                             max(n for n, _ in cuts) if longest is None else longest, st, out, H, d, e, EPS)
+                             max(n for n, _ in cuts) if longest is None else longest, st, out, H, d, e, EPS, rope=rope)
     ud = u.double()
     want, left_behind = torch.zeros(T, H * e, dtype=torch.float64), slots.double().clone()
     for t0, n, before, slot in segs.tolist():
