@@ -1,7 +1,9 @@
 """A paged-KV inference engine for one B200: Qwen3 dense decoder, Surelorn
 (latent attention, routed experts), Bumisun (windowed attention with sinks beside
-Mamba-2 layers, clamped experts) and Pamarax (gated attention with normed q/k, matrix
-LSTM layers, attention beside a gated delta rule), token ids in, token ids out.
+Mamba-2 layers, clamped experts), Pamarax (gated attention with normed q/k, matrix
+LSTM layers, attention beside a gated delta rule), Tebozen (differential attention,
+matrix LSTM, latent attention, squared-relu experts) and Reperax (retention, chunked
+attention beside gated linear attention, layers run in passes), token ids in, token ids out.
 
     from paged_llm_rs_b200 import Engine
     engine = Engine("model_dir", dtype="bfloat16")

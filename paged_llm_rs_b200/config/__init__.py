@@ -5,3 +5,4 @@ from .surelorn import SurelornConfig
 from .bumisun import BumisunConfig
 from .pamarax import PamaraxConfig
 from .tebozen import TebozenConfig
+from .reperax import ReperaxConfig
