@@ -2,8 +2,10 @@
 (latent attention, routed experts), Bumisun (windowed attention with sinks beside
 Mamba-2 layers, clamped experts), Pamarax (gated attention with normed q/k, matrix
 LSTM layers, attention beside a gated delta rule), Tebozen (differential attention,
-matrix LSTM, latent attention, squared-relu experts) and Reperax (retention, chunked
-attention beside gated linear attention, layers run in passes), token ids in, token ids out.
+matrix LSTM, latent attention, squared-relu experts), Reperax (retention, chunked
+attention beside gated linear attention, layers run in passes) and Tubevik (windowed
+attention over lent keys, chunked attention beside a gated delta rule with a decay a key
+entry, sublayers side by side), token ids in, token ids out.
 
     from paged_llm_rs_b200 import Engine
     engine = Engine("model_dir", dtype="bfloat16")

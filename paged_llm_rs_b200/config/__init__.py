@@ -6,3 +6,4 @@ from .bumisun import BumisunConfig
 from .pamarax import PamaraxConfig
 from .tebozen import TebozenConfig
 from .reperax import ReperaxConfig
+from .tubevik import TubevikConfig

@@ -13,6 +13,8 @@
 //                      rather than wait for the CTA that has it.
 //   poly_norm          y = a N(u) + b N(u^2) + c N(u^3) + e, N(z) = z / sqrt(mean(z^2) + eps) over a row, powers entry by entry
 //   softcap32          x = cap tanh(x / cap)
+//   add_terms_norm32   x += c1 d1 + c2 d2 + c3 d3 (in place; terms may be absent), y = norm(x): the root mean square's or, with
+//                      the mean taken off first, a layer norm with a bias.  What a block does whose sublayers read ONE norm.
 //
 // Norms, gates, sums and the shift are float whatever the compute dtype; each output is rounded once.
 #include "matrix_memory.cuh"
@@ -272,6 +274,122 @@ PLLM_EXPORT int pllm_gated_sum_norm32(int dtype, const float* x, const void* a1,
             launch_chained(gated_sum_norm32_kernel<T, N>, dim3(grid), dim3(threads), smem, stream, g, x_out, gain1, (T*)y1, shift, (T*)ys, gain2, \
                            (T*)y2, (const MMSegment*)segs, n_segs, state, state_stride, rows, n_rows, width, eps, run); } while (0)
         if (vec) GS_LAUNCH(V); else GS_LAUNCH(1);
+    });
+    return launch_status();
+}
+
+// Up to three terms a stream still has to take: rows of the compute dtype with strides in elements, a constant each.
+#define GS_TERMS 3
+struct StreamTerms {
+    const void* d[GS_TERMS];
+    float c[GS_TERMS];
+    int stride[GS_TERMS];
+};
+
+// A CTA a row; a thread has the same entries of it in every pass, N at a time: the first ones in registers, the others in
+// shared memory.  The sum is stored only when every row is taken (rows null).  bias null and centered 0: the root mean square's
+// norm; centered: (x - mean) / sqrt(mean of squared deviations + eps).
+template <typename T, int N>
+__global__ void __launch_bounds__(512) add_terms_norm32_kernel(float* x, StreamTerms terms, const float* __restrict__ gain, const float* __restrict__ bias,
+                                                               int centered, T* __restrict__ y, const int* __restrict__ rows, int width, float eps) {
+    extern __shared__ __align__(16) float gs_smem[];          // [width - blockDim.x N]: what the registers do not hold
+    __shared__ float scratch[32];
+    const int stride = blockDim.x * N, c0 = threadIdx.x * N;
+    float w0[N], b0[N];
+    const bool some = c0 < width;
+    if (some) {                                               // the weights do not come from the kernel before
+        gs_load32<N>(gain + c0, w0);
+        if (bias) gs_load32<N>(bias + c0, b0);
+    }
+    pdl_launch_dependents();
+    pdl_wait(KID_GATED_STREAM);
+    const size_t r = rows ? (size_t)rows[blockIdx.x] : (size_t)blockIdx.x;
+    float* xr = x + r * width;
+    const bool store = terms.d[0] != nullptr && rows == nullptr;
+    float keep[N];
+    float sum = 0.f, ss = 0.f;
+    for (int c = c0; c < width; c += stride) {
+        float v[N];
+        gs_load32<N>(xr + c, v);
+#pragma unroll
+        for (int i = 0; i < GS_TERMS; i++) {
+            if (!terms.d[i]) break;
+            float t[N];
+            gs_load<T, N>((const T*)terms.d[i] + r * terms.stride[i] + c, t);
+#pragma unroll
+            for (int k = 0; k < N; k++) v[k] = fmaf(terms.c[i], t[k], v[k]);
+        }
+        if (store) gs_store32<N>(xr + c, v);
+#pragma unroll
+        for (int k = 0; k < N; k++) { sum += v[k]; ss = fmaf(v[k], v[k], ss); }
+        if (c == c0) {
+#pragma unroll
+            for (int k = 0; k < N; k++) keep[k] = v[k];
+        } else {
+            gs_store32<N>(gs_smem + c - stride, v);
+        }
+    }
+    float mean = 0.f;
+    if (centered) {
+        mean = block_sum(sum, scratch) / (float)width;
+        ss = 0.f;
+        for (int c = c0; c < width; c += stride) {
+            float v[N];
+            if (c == c0) {
+#pragma unroll
+                for (int k = 0; k < N; k++) v[k] = keep[k];
+            } else {
+                gs_load32<N>(gs_smem + c - stride, v);
+            }
+#pragma unroll
+            for (int k = 0; k < N; k++) { const float o = v[k] - mean; ss = fmaf(o, o, ss); }
+        }
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)width + eps);
+    T* yr = y + (size_t)blockIdx.x * width;
+    for (int c = c0; c < width; c += stride) {
+        float v[N], w[N], b[N];
+        if (c == c0) {
+#pragma unroll
+            for (int k = 0; k < N; k++) { v[k] = keep[k]; w[k] = w0[k]; b[k] = bias ? b0[k] : 0.f; }
+        } else {
+            gs_load32<N>(gs_smem + c - stride, v);
+            gs_load32<N>(gain + c, w);
+            if (bias) gs_load32<N>(bias + c, b);
+            else {
+#pragma unroll
+                for (int k = 0; k < N; k++) b[k] = 0.f;
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < N; k++) v[k] = fmaf((v[k] - mean) * inv, w[k], b[k]);
+        gs_store<T, N>(yr + c, v);
+    }
+}
+
+// Terms from the first on; an absent one ends them.  With `rows` (n_rows of them) only those rows are formed and normed, into
+// row i of y, and x stays as it is.
+PLLM_EXPORT int pllm_add_terms_norm32(int dtype, float* x, const void* d1, int s1, float c1, const void* d2, int s2, float c2, const void* d3, int s3,
+                                      float c3, const float* gain, const float* bias, int centered, void* y, const int* rows, int n_rows, int width,
+                                      float eps, cudaStream_t stream) {
+    if (n_rows <= 0) return PLLM_OK;
+    if (width <= 0 || !x || !gain || !y || (d2 && !d1) || (d3 && !d2)) return PLLM_ERR_SIZE;
+    StreamTerms terms = {{d1, d2, d3}, {c1, c2, c3}, {s1, s2, s3}};
+    PLLM_DISPATCH_DTYPE(dtype, {
+        constexpr int V = Vec16<T>::N;
+        const uintptr_t p = (uintptr_t)x | (uintptr_t)d1 | (uintptr_t)d2 | (uintptr_t)d3 | (uintptr_t)gain | (uintptr_t)bias | (uintptr_t)y;
+        const bool vec = width % V == 0 && (p & 15) == 0 && (!d1 || s1 % V == 0) && (!d2 || s2 % V == 0) && (!d3 || s3 % V == 0);
+        // four entries a thread at the least where the dtype's vectors are four, eight else; rows of few vectors in small CTAs
+        const int per = vec ? V : 1;
+        int threads = ((width + per - 1) / per + 31) / 32 * 32;
+        if (threads > 512) threads = 512;
+        const int held = threads * per;
+        const size_t smem = width > held ? (size_t)(width - held) * sizeof(float) : 0;
+        if (smem > 200 * 1024) return PLLM_ERR_LIMIT;
+        auto kernel = vec ? add_terms_norm32_kernel<T, V> : add_terms_norm32_kernel<T, 1>;
+        if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        launch_chained(kernel, dim3(n_rows), dim3(threads), smem, stream, x, terms, gain, bias, centered, (T*)y, rows, width, eps);
     });
     return launch_status();
 }

@@ -131,65 +131,6 @@ PLLM_EXPORT int pllm_rope_table(const int* positions, const float* inv_freq, flo
     return launch_status();
 }
 
-// two float products, or multiply-adds, in one instruction
-typedef unsigned long long f32x2;
-__device__ __forceinline__ f32x2 la_pair(float x, float y) {
-    f32x2 r;
-    asm("mov.b64 %0, {%1, %2};\n" : "=l"(r) : "f"(x), "f"(y));
-    return r;
-}
-__device__ __forceinline__ float2 la_unpair(f32x2 v) {
-    float2 r;
-    asm("mov.b64 {%0, %1}, %2;\n" : "=f"(r.x), "=f"(r.y) : "l"(v));
-    return r;
-}
-__device__ __forceinline__ f32x2 la_mul2(f32x2 a, f32x2 b) {
-    f32x2 r;
-    asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(r) : "l"(a), "l"(b));
-    return r;
-}
-__device__ __forceinline__ f32x2 la_fma2(f32x2 a, f32x2 b, f32x2 c) {
-    f32x2 r;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-    return r;
-}
-
-// Block w of the step: the segments' blocks of L tokens one after the other.
-struct LABlock {
-    int seg, tb, blocks;       // segment, which of its blocks, how many it has (seg -1: no such block)
-    int rank;                  // its index among the blocks of segments of several blocks
-};
-__device__ __forceinline__ LABlock la_find_block(const MMSegment* __restrict__ segs, int n_segs, int w, int L) {
-    const int lane = threadIdx.x & 31;
-    int seen = 0, several = 0;
-    for (int base = 0; base < n_segs; base += 32) {
-        const int c = base + lane < n_segs ? segs[base + lane].count : 0;
-        const int nb = c > 0 ? (c + L - 1) / L : 0, mb = nb > 1 ? nb : 0;
-        int sum = nb, msum = mb;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const int x = __shfl_up_sync(0xffffffffu, sum, o), y = __shfl_up_sync(0xffffffffu, msum, o);
-            if (lane >= o) { sum += x; msum += y; }
-        }
-        const int first = seen + sum - nb;
-        const unsigned hit = __ballot_sync(0xffffffffu, w >= first && w < first + nb);
-        if (hit) {
-            const int src = __ffs(hit) - 1;
-            LABlock b;
-            b.seg = base + src;
-            b.tb = w - __shfl_sync(0xffffffffu, first, src);
-            b.blocks = __shfl_sync(0xffffffffu, nb, src);
-            b.rank = several + __shfl_sync(0xffffffffu, msum - mb, src) + b.tb;
-            return b;
-        }
-        seen += __shfl_sync(0xffffffffu, sum, 31);
-        several += __shfl_sync(0xffffffffu, msum, 31);
-    }
-    LABlock none;
-    none.seg = -1; none.tb = none.blocks = none.rank = 0;
-    return none;
-}
-
 // grid (blocks, heads, slices of e).  u: [tokens, u_stride] of the compute dtype; alpha: [tokens, H d] float (per entry).
 template <typename T, int NPT, bool CHANNEL>
 __global__ void __launch_bounds__(256, 2) la_scan_kernel(const T* u, LAShape sh, const float2* rope, const float* alpha, const MMSegment* __restrict__ segs, int n_segs,
@@ -208,7 +149,7 @@ __global__ void __launch_bounds__(256, 2) la_scan_kernel(const T* u, LAShape sh,
     float* y_s = v_s + ck * Ps;                             // [ck][parts][Ps]
     pdl_launch_dependents();
     pdl_wait(KID_LINEAR_ATT);
-    const LABlock b = la_find_block(segs, n_segs, blockIdx.x, L);
+    const MMBlock b = mm_find_block(segs, n_segs, blockIdx.x, L);
     if (b.seg < 0) return;
     const MMSegment s = segs[b.seg];
     const int h = blockIdx.y, p0 = blockIdx.z * Ps, tid = threadIdx.x;
@@ -226,7 +167,7 @@ __global__ void __launch_bounds__(256, 2) la_scan_kernel(const T* u, LAShape sh,
         for (int c = 0; c < LA_COLS; c++) {
             const float* p = S + (size_t)n * E + e + c;
             const bool in = from && e + c < E;
-            st[c][k / 2] = la_pair((in && n < d) ? p[0] : 0.f, (in && n + 1 < d) ? p[E] : 0.f);
+            st[c][k / 2] = mm_pair((in && n < d) ? p[0] : 0.f, (in && n + 1 < d) ? p[E] : 0.f);
         }
     }
     // A constant decay that is not too strong leaves the token loop: a chunk's state is kept over decay^(t + 1), so that values
@@ -330,12 +271,12 @@ __global__ void __launch_bounds__(256, 2) la_scan_kernel(const T* u, LAShape sh,
             }
         }
         if (part < parts) {
-            const f32x2 dd = la_pair(decay, decay);
-            const f32x2 zero = la_pair(0.f, 0.f);
+            const f32x2 dd = mm_pair(decay, decay);
+            const f32x2 zero = mm_pair(0.f, 0.f);
 #define LA_TOKENS(UPDATE) do { \
             for (int t = 0; t < nt; t++) { \
                 const float4 v4 = *reinterpret_cast<const float4*>(v_s + t * Ps + col); \
-                const f32x2 v[LA_COLS] = {la_pair(v4.x, v4.x), la_pair(v4.y, v4.y), la_pair(v4.z, v4.z), la_pair(v4.w, v4.w)}; \
+                const f32x2 v[LA_COLS] = {mm_pair(v4.x, v4.x), mm_pair(v4.y, v4.y), mm_pair(v4.z, v4.z), mm_pair(v4.w, v4.w)}; \
                 const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(k_s + t * NP + part * NPT); \
                 const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(q_s + t * NP + part * NPT); \
                 const ulonglong2* a4 = reinterpret_cast<const ulonglong2*>(a_s + t * NP + part * NPT); \
@@ -349,23 +290,23 @@ __global__ void __launch_bounds__(256, 2) la_scan_kernel(const T* u, LAShape sh,
                     _Pragma("unroll") \
                     for (int c = 0; c < LA_COLS; c++) { \
                         UPDATE; \
-                        acc[c] = la_fma2(st[c][2 * k], qv.x, acc[c]); acc[c] = la_fma2(st[c][2 * k + 1], qv.y, acc[c]); \
+                        acc[c] = mm_fma2(st[c][2 * k], qv.x, acc[c]); acc[c] = mm_fma2(st[c][2 * k + 1], qv.y, acc[c]); \
                     } \
                 } \
-                const float2 r0 = la_unpair(acc[0]), r1 = la_unpair(acc[1]), r2 = la_unpair(acc[2]), r3 = la_unpair(acc[3]); \
+                const float2 r0 = mm_unpair(acc[0]), r1 = mm_unpair(acc[1]), r2 = mm_unpair(acc[2]), r3 = mm_unpair(acc[3]); \
                 *reinterpret_cast<float4*>(y_s + (t * parts + part) * Ps + col) = make_float4(r0.x + r0.y, r1.x + r1.y, r2.x + r2.y, r3.x + r3.y); \
             } } while (0)
             if (scaled)
-                LA_TOKENS(st[c][2 * k] = la_fma2(kv.x, v[c], st[c][2 * k]); st[c][2 * k + 1] = la_fma2(kv.y, v[c], st[c][2 * k + 1]));
+                LA_TOKENS(st[c][2 * k] = mm_fma2(kv.x, v[c], st[c][2 * k]); st[c][2 * k + 1] = mm_fma2(kv.y, v[c], st[c][2 * k + 1]));
             else
-                LA_TOKENS(st[c][2 * k] = la_fma2(av.x, st[c][2 * k], la_mul2(kv.x, v[c]));
-                          st[c][2 * k + 1] = la_fma2(av.y, st[c][2 * k + 1], la_mul2(kv.y, v[c])));
+                LA_TOKENS(st[c][2 * k] = mm_fma2(av.x, st[c][2 * k], mm_mul2(kv.x, v[c]));
+                          st[c][2 * k + 1] = mm_fma2(av.y, st[c][2 * k + 1], mm_mul2(kv.y, v[c])));
             if (scaled) {
-                const f32x2 f = la_pair(pow_s[nt - 1], pow_s[nt - 1]);
+                const f32x2 f = mm_pair(pow_s[nt - 1], pow_s[nt - 1]);
 #pragma unroll
                 for (int c = 0; c < LA_COLS; c++)
 #pragma unroll
-                    for (int k = 0; k < NPT / 2; k++) st[c][k] = la_mul2(st[c][k], f);
+                    for (int k = 0; k < NPT / 2; k++) st[c][k] = mm_mul2(st[c][k], f);
             }
         }
         __syncthreads();
@@ -398,7 +339,7 @@ __global__ void __launch_bounds__(256, 2) la_scan_kernel(const T* u, LAShape sh,
 #pragma unroll
             for (int c = 0; c < LA_COLS; c++) {
                 if (e + c >= E) break;
-                const float2 x = la_unpair(st[c][k / 2]);
+                const float2 x = mm_unpair(st[c][k / 2]);
                 if (n < d) dst[(size_t)n * E + e + c] = x.x;
                 if (n + 1 < d) dst[(size_t)(n + 1) * E + e + c] = x.y;
             }
@@ -453,7 +394,7 @@ __global__ void __launch_bounds__(256) la_block_outputs_kernel(const MMSegment* 
     __shared__ __align__(16) float S_s[LA_TK][LA_TC];
     pdl_launch_dependents();
     pdl_wait(KID_LINEAR_ATT);
-    const LABlock b = la_find_block(segs, n_segs, blockIdx.x, L);
+    const MMBlock b = mm_find_block(segs, n_segs, blockIdx.x, L);
     if (b.seg < 0 || b.tb == 0) return;
     const MMSegment s = segs[b.seg];
     const int h = blockIdx.y / col_tiles, c0 = (blockIdx.y % col_tiles) * LA_TC, t0 = blockIdx.z * LA_TT;
@@ -465,7 +406,7 @@ __global__ void __launch_bounds__(256) la_block_outputs_kernel(const MMSegment* 
     const bool vec = E % 4 == 0;
     f32x2 acc[4][2];
 #pragma unroll
-    for (int r = 0; r < 4; r++) acc[r][0] = acc[r][1] = la_pair(0.f, 0.f);
+    for (int r = 0; r < 4; r++) acc[r][0] = acc[r][1] = mm_pair(0.f, 0.f);
     for (int k0 = 0; k0 < d; k0 += LA_TK) {
         __syncthreads();
 #pragma unroll
@@ -497,8 +438,8 @@ __global__ void __launch_bounds__(256) la_block_outputs_kernel(const MMSegment* 
             const float qq[4] = {qv.x, qv.y, qv.z, qv.w};
 #pragma unroll
             for (int r = 0; r < 4; r++) {
-                const f32x2 q2 = la_pair(qq[r], qq[r]);
-                acc[r][0] = la_fma2(q2, sv.x, acc[r][0]); acc[r][1] = la_fma2(q2, sv.y, acc[r][1]);
+                const f32x2 q2 = mm_pair(qq[r], qq[r]);
+                acc[r][0] = mm_fma2(q2, sv.x, acc[r][0]); acc[r][1] = mm_fma2(q2, sv.y, acc[r][1]);
             }
         }
     }
@@ -507,7 +448,7 @@ __global__ void __launch_bounds__(256) la_block_outputs_kernel(const MMSegment* 
         const int t = ty * 4 + r, c = c0 + tx * 4;
         if (t >= nt) continue;
         float* yr = y + (tok0 + t) * H * E + (size_t)h * E + c;
-        const float2 x0 = la_unpair(acc[r][0]), x1 = la_unpair(acc[r][1]);
+        const float2 x0 = mm_unpair(acc[r][0]), x1 = mm_unpair(acc[r][1]);
         if (c < E) yr[0] += x0.x;
         if (c + 1 < E) yr[1] += x0.y;
         if (c + 2 < E) yr[2] += x1.x;

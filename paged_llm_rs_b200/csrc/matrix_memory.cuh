@@ -1,5 +1,5 @@
-// What the recurrences with a matrix of state a head share: a step's segments, loads of 16 bytes as floats, and the head
-// norm with its gate behind a recurrence.
+// What the recurrences with a matrix of state a head share: a step's segments and where a segment's blocks of tokens lie, loads
+// of 16 bytes as floats, products of two floats in one instruction, and the head norm with its gate behind a recurrence.
 #pragma once
 
 #include "common.cuh"
@@ -27,6 +27,65 @@ __device__ __forceinline__ void mm_fetch16(const bf16* p, float* dst, float scal
                                                   __uint_as_float(r.y << 16) * scale, __uint_as_float(r.y & 0xffff0000u) * scale);
     *reinterpret_cast<float4*>(dst + 4) = make_float4(__uint_as_float(r.z << 16) * scale, __uint_as_float(r.z & 0xffff0000u) * scale,
                                                       __uint_as_float(r.w << 16) * scale, __uint_as_float(r.w & 0xffff0000u) * scale);
+}
+
+// two float products, or multiply-adds, in one instruction
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 mm_pair(float x, float y) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};\n" : "=l"(r) : "f"(x), "f"(y));
+    return r;
+}
+__device__ __forceinline__ float2 mm_unpair(f32x2 v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;\n" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ f32x2 mm_mul2(f32x2 a, f32x2 b) {
+    f32x2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ f32x2 mm_fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+
+// Block w of the step: the segments' blocks of L tokens one after the other.
+struct MMBlock {
+    int seg, tb, blocks;       // segment, which of its blocks, how many it has (seg -1: no such block)
+    int rank;                  // its index among the blocks of segments of several blocks
+};
+__device__ __forceinline__ MMBlock mm_find_block(const MMSegment* __restrict__ segs, int n_segs, int w, int L) {
+    const int lane = threadIdx.x & 31;
+    int seen = 0, several = 0;
+    for (int base = 0; base < n_segs; base += 32) {
+        const int c = base + lane < n_segs ? segs[base + lane].count : 0;
+        const int nb = c > 0 ? (c + L - 1) / L : 0, mb = nb > 1 ? nb : 0;
+        int sum = nb, msum = mb;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int x = __shfl_up_sync(0xffffffffu, sum, o), y = __shfl_up_sync(0xffffffffu, msum, o);
+            if (lane >= o) { sum += x; msum += y; }
+        }
+        const int first = seen + sum - nb;
+        const unsigned hit = __ballot_sync(0xffffffffu, w >= first && w < first + nb);
+        if (hit) {
+            const int src = __ffs(hit) - 1;
+            MMBlock b;
+            b.seg = base + src;
+            b.tb = w - __shfl_sync(0xffffffffu, first, src);
+            b.blocks = __shfl_sync(0xffffffffu, nb, src);
+            b.rank = several + __shfl_sync(0xffffffffu, msum - mb, src) + b.tb;
+            return b;
+        }
+        seen += __shfl_sync(0xffffffffu, sum, 31);
+        several += __shfl_sync(0xffffffffu, msum, 31);
+    }
+    MMBlock none;
+    none.seg = -1; none.tb = none.blocks = none.rank = 0;
+    return none;
 }
 
 // A warp a (token, head): o / rms(o) * gain * act(gate).  y float [tokens, H e]; gate: [tokens, g_stride] of the compute dtype;

@@ -2,18 +2,21 @@
 // queries and keys, and the gate on an attention's output.
 //
 //   normed_qk_kv_write   one pass over the stacked projection [q | k | (v) | ...] of the step's tokens, a CTA a token:
+//                          biases on q, k and v (each may be absent)
 //                          norm      0 none; 1 each head by its own root mean square, one gain of dk entries shared by the
 //                                    heads; 2 the whole projection (all heads of q, and likewise of k) by one root mean
-//                                    square, a gain of its full size
+//                                    square, a gain of its full size; 3 each head by its own root mean square as it is behind
+//                                    the rotation, no gain
 //                          q *= 1 + coef * ln(floor((p + 1) / every) + 1)     (every = 0: no such factor)
-//                          rotation of the first `rot` entries of every q and k head, entry i with entry i + rot / 2, by the
-//                                    angle p * inv_freq[i], a float product
+//                          rotation of the first `rot` entries of every q and k head, entry i with entry i + rot / 2 or entry
+//                                    2i with entry 2i + 1, by the angle p * inv_freq[i], a float product; cos and sin times a
+//                                    factor
 //                          q to its own tensor; k | v to the token's row of the joined pool; v is the projection's v
 //                          part, or (values_are_keys) the raw key projection, neither normed nor rotated
 //                        Everything is float from the projection's values to the one rounding on the way out.
 //   gate_mul             y[t, c] *= sigmoid(g[t, c / per]) (kind 0) or silu(g[t, c / per]) (kind 1); g rows may be strided; per 1: a
 //                        gate an entry, per = a head's size: a gate a head
-#include "common.cuh"
+#include "matrix_memory.cuh"
 
 enum : int { KID_NORMED_QK = 90 };
 
@@ -22,114 +25,180 @@ __device__ __forceinline__ float nq_sigmoid(float z) { return 1.0f / (1.0f + exp
 // Sum over the CTA, for every thread (scratch: 32 floats).
 __device__ __forceinline__ float nq_block_sum(float v, float* scratch) { return block_sum(v, scratch); }
 
-template <typename T>
-__global__ void __launch_bounds__(256) normed_qk_kv_write_kernel(const T* proj, int row_stride, int k_off, int v_off, T* __restrict__ q_out,
-                                                                 const float* __restrict__ q_gain, const float* __restrict__ k_gain,
-                                                                 int norm, float eps, float temp_coef, int temp_every,
-                                                                 const float* __restrict__ inv_freq, int rot,
+// What the pass over a token's projection does.
+struct NormedQK {
+    int k_off, v_off;                // columns of the keys and the values (k_off negative: queries only)
+    const float *q_bias, *k_bias, *v_bias;       // nh dk, nkv dk, nkv dv (null: none)
+    const float *q_gain, *k_gain;
+    int norm;                        // 0 none; 1 a head; 2 the whole projection; 3 a head, behind the rotation, no gain
+    float eps;
+    float temp_coef;
+    int temp_every;
+    const float* inv_freq;
+    int rot;                         // leading entries of each head that turn
+    int pairs;                       // 0: entry i turns with entry i + rot / 2; 1: entry 2i with entry 2i + 1
+    float rot_factor;                // on cos and sin
+    int nh, nkv, dk, dv, values_are_keys, page_size;
+    long long pool_rows;
+};
+
+// entry e of a head that lies in shared memory, normed and turned
+__device__ __forceinline__ float nq_entry(const float* head, const float* __restrict__ gain, int e, float inv, const NormedQK& a, const float2* turn) {
+    float v = head[e] * inv;
+    if (gain) v *= gain[e];
+    if (e < a.rot) {
+        const int half = a.rot >> 1;
+        const bool first = a.pairs ? !(e & 1) : e < half;
+        const int f = a.pairs ? e >> 1 : (first ? e : e - half);
+        const int j = a.pairs ? e ^ 1 : (first ? e + half : e - half);
+        float other = head[j] * inv;
+        if (gain) other *= gain[j];
+        const float2 t = turn[f];
+        v = first ? v * t.x - other * t.y : v * t.x + other * t.y;
+    }
+    return v;
+}
+
+// A CTA a token.  Its queries and keys lie in shared memory as floats; the cos and sin of its angles are formed once for all heads.
+// N: entries a thread takes at a time (4 where every part and head is whole groups of four, else 1).
+template <typename T, int N>
+__global__ void __launch_bounds__(256) normed_qk_kv_write_kernel(const T* proj, int row_stride, NormedQK a, T* __restrict__ q_out,
                                                                  const int* __restrict__ positions, const int* __restrict__ slots,
-                                                                 T* kv_pool, int nh, int nkv, int dk, int dv, int values_are_keys,
-                                                                 int page_size, long long pool_rows, int* status) {
-    extern __shared__ float nq_smem[];
-    float* head_inv = nq_smem;            // [nh + nkv] 1 / rms of each head (norm 1)
+                                                                 T* kv_pool, int* status) {
+    extern __shared__ __align__(16) float nq_smem[];
+    const int nh = a.nh, nkv = a.k_off >= 0 ? a.nkv : 0, dk = a.dk, dv = a.dv;
+    const int qw = nh * dk, kw = nkv * dk;
+    float* q_s = nq_smem;                                     // [qw]
+    float* k_s = q_s + (qw + 3) / 4 * 4;                      // [kw]
+    float2* turn = reinterpret_cast<float2*>(k_s + (kw + 3) / 4 * 4);      // [rot / 2] cos and sin times the factor
+    float* head_inv = reinterpret_cast<float*>(turn + a.rot / 2);          // [nh + nkv] 1 / rms of each head (norms 1 and 3)
     __shared__ float scratch[32];
     pdl_launch_dependents();
-    pdl_wait(KID_NORMED_QK);
+    // (the step's packed buffer is in place before the kernels of the step begin)
     const int t = blockIdx.x;
-    const T* row = proj + (size_t)t * row_stride;
-    const T* kr = row + k_off;
     const int pos = positions[t];
-    const float p = (float)pos;
-    const int half = rot / 2;
-    const int qw = nh * dk, kw = nkv * dk;
-    float q_inv = 1.f, k_inv = 1.f;
-    if (norm == 2) {
-        float sq = 0.f, sk = 0.f;
-        for (int i = threadIdx.x; i < qw; i += blockDim.x) { const float v = to_f32(row[i]); sq += v * v; }
-        for (int i = threadIdx.x; i < kw; i += blockDim.x) { const float v = to_f32(kr[i]); sk += v * v; }
-        sq = nq_block_sum(sq, scratch);
-        sk = nq_block_sum(sk, scratch);
-        q_inv = 1.0f / sqrtf(sq / (float)qw + eps);
-        k_inv = 1.0f / sqrtf(sk / (float)kw + eps);
-    } else if (norm == 1) {
-        const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-        for (int h = warp; h < nh + nkv; h += warps) {
-            const T* hr = h < nh ? row + (size_t)h * dk : kr + (size_t)(h - nh) * dk;
-            float s = 0.f;
-            for (int e = lane; e < dk; e += 32) { const float v = to_f32(hr[e]); s += v * v; }
-            s = warp_sum(s);
-            if (lane == 0) head_inv[h] = 1.0f / sqrtf(s / (float)dk + eps);
+    const int slot = slots ? slots[t] : -1;
+    for (int f = threadIdx.x; f < a.rot / 2; f += blockDim.x) {
+        float s, c;
+        sincosf((float)pos * a.inv_freq[f], &s, &c);
+        turn[f] = make_float2(c * a.rot_factor, s * a.rot_factor);
+    }
+    pdl_wait(KID_NORMED_QK);
+    const T* row = proj + (size_t)t * row_stride;
+    const T* kr = row + a.k_off;
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x * N; i < qw; i += blockDim.x * N) {
+        float v[N];
+        if constexpr (N == 4) head_quad_load(row + i, v); else v[0] = to_f32(row[i]);
+#pragma unroll
+        for (int k = 0; k < N; k++) {
+            if (a.q_bias) v[k] += a.q_bias[i + k];
+            q_s[i + k] = v[k];
+            sq = fmaf(v[k], v[k], sq);
         }
+    }
+    for (int i = threadIdx.x * N; i < kw; i += blockDim.x * N) {
+        float v[N];
+        if constexpr (N == 4) head_quad_load(kr + i, v); else v[0] = to_f32(kr[i]);
+#pragma unroll
+        for (int k = 0; k < N; k++) {
+            if (a.k_bias) v[k] += a.k_bias[i + k];
+            k_s[i + k] = v[k];
+            sk = fmaf(v[k], v[k], sk);
+        }
+    }
+    float q_inv = 1.f, k_inv = 1.f;
+    if (a.norm == 2) {
+        sq = nq_block_sum(sq, scratch);
+        q_inv = 1.0f / sqrtf(sq / (float)qw + a.eps);
+        if (kw) {
+            sk = nq_block_sum(sk, scratch);
+            k_inv = 1.0f / sqrtf(sk / (float)kw + a.eps);
+        }
+    } else {
         __syncthreads();
+        if (a.norm) {
+            // (a pair keeps its length when it turns, but for the factor: a head's mean square behind the rotation follows from
+            // the entries ahead of it)
+            const float turned = a.norm == 3 ? a.rot_factor * a.rot_factor : 1.f;
+            const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+            for (int h = warp; h < nh + nkv; h += warps) {
+                const float* hr = h < nh ? q_s + h * dk : k_s + (h - nh) * dk;
+                float s = 0.f;
+                for (int e = lane; e < dk; e += 32) { const float v = hr[e]; s = fmaf(e < a.rot ? v * turned : v, v, s); }
+                s = warp_sum(s);
+                if (lane == 0) head_inv[h] = 1.0f / sqrtf(s / (float)dk + a.eps);
+            }
+            __syncthreads();
+        }
     }
     float temp = 1.f;
-    if (temp_every > 0) temp = 1.0f + temp_coef * logf((float)((pos + 1) / temp_every + 1));
-    // queries
+    if (a.temp_every > 0) temp = 1.0f + a.temp_coef * logf((float)((pos + 1) / a.temp_every + 1));
+    const bool a_head = a.norm == 1 || a.norm == 3;
+    const int gain_stride = a.norm == 2 ? dk : 0;             // a gain of the projection's size, or one a head shared by the heads
     T* qo = q_out + (size_t)t * qw;
-    for (int i = threadIdx.x; i < qw; i += blockDim.x) {
-        const int h = i / dk, e = i % dk;
-        const float inv = norm == 2 ? q_inv : norm == 1 ? head_inv[h] : 1.f;
-        float v = to_f32(row[i]) * inv;
-        if (norm) v *= q_gain[norm == 2 ? i : e];
-        if (e < rot) {
-            const int f = e < half ? e : e - half;
-            const int j = e < half ? i + half : i - half;
-            float s, c;
-            sincosf(p * inv_freq[f], &s, &c);
-            float other = to_f32(row[j]) * inv;
-            if (norm) other *= q_gain[norm == 2 ? j : (e < half ? e + half : e - half)];
-            v = e < half ? v * c - other * s : v * c + other * s;
-        }
-        qo[i] = from_f32<T>(v * temp);
+    for (int i = threadIdx.x * N; i < qw; i += blockDim.x * N) {
+        const int h = i / dk, e = i - h * dk;
+        const float inv = a_head ? head_inv[h] : q_inv;
+        const float* g = a.q_gain ? a.q_gain + h * gain_stride : nullptr;
+        float v[N];
+#pragma unroll
+        for (int k = 0; k < N; k++) v[k] = nq_entry(q_s + h * dk, g, e + k, inv, a, turn) * temp;
+        if constexpr (N == 4) head_quad_store(qo + i, v); else qo[i] = from_f32<T>(v[0]);
     }
-    const int slot = slots ? slots[t] : -1;
-    if (kv_pool == nullptr || slot < 0) return;
-    if ((long long)slot >= pool_rows) { if (threadIdx.x == 0) atomicOr(status, 2); return; }
-    const int page = slot / page_size, off = slot % page_size;
+    if (kv_pool == nullptr || slot < 0 || nkv == 0) return;
+    if ((long long)slot >= a.pool_rows) { if (threadIdx.x == 0) atomicOr(status, 2); return; }
+    const int page = slot / a.page_size, off = slot % a.page_size;
     const int w = dk + dv;
-    const T* vr = row + v_off;
-    for (int i = threadIdx.x; i < nkv * w; i += blockDim.x) {
-        const int g = i / w, e = i % w;
-        T* dst = kv_pool + (((size_t)page * nkv + g) * page_size + off) * w;
-        if (e >= dk) {
-            // a value: copied as it is (the raw key projection, or the projection's own value)
-            dst[e] = values_are_keys ? kr[g * dk + e - dk] : vr[g * dv + e - dk];
-            continue;
+    const T* vr = row + a.v_off;
+    for (int i = threadIdx.x * N; i < nkv * w; i += blockDim.x * N) {
+        const int g = i / w, e = i - g * w;
+        T* dst = kv_pool + (((size_t)page * nkv + g) * a.page_size + off) * w + e;
+        float v[N];
+        if (e < dk) {
+            const float inv = a_head ? head_inv[nh + g] : k_inv;
+            const float* gn = a.k_gain ? a.k_gain + g * gain_stride : nullptr;
+#pragma unroll
+            for (int k = 0; k < N; k++) v[k] = nq_entry(k_s + g * dk, gn, e + k, inv, a, turn);
+        } else if (a.values_are_keys) {
+            // the raw key projection, neither normed nor turned
+#pragma unroll
+            for (int k = 0; k < N; k++) v[k] = k_s[g * dk + e - dk + k];
+        } else {
+            const int c = g * dv + e - dk;
+            if constexpr (N == 4) head_quad_load(vr + c, v); else v[0] = to_f32(vr[c]);
+            if (a.v_bias) {
+#pragma unroll
+                for (int k = 0; k < N; k++) v[k] += a.v_bias[c + k];
+            }
         }
-        const int ki = g * dk + e;
-        const float inv = norm == 2 ? k_inv : norm == 1 ? head_inv[nh + g] : 1.f;
-        float v = to_f32(kr[ki]) * inv;
-        if (norm) v *= k_gain[norm == 2 ? ki : e];
-        if (e < rot) {
-            const int f = e < half ? e : e - half;
-            const int j = e < half ? ki + half : ki - half;
-            float s, c;
-            sincosf(p * inv_freq[f], &s, &c);
-            float other = to_f32(kr[j]) * inv;
-            if (norm) other *= k_gain[norm == 2 ? j : (e < half ? e + half : e - half)];
-            v = e < half ? v * c - other * s : v * c + other * s;
-        }
-        dst[e] = from_f32<T>(v);
+        if constexpr (N == 4) head_quad_store(dst, v); else dst[0] = from_f32<T>(v[0]);
     }
 }
 
-// proj: [tokens, row_stride] with q at 0, k at k_off, v at v_off (ignored when values_are_keys, which needs dv == dk).
-// q_gain / k_gain: float, dk entries (norm 1) or nh * dk and nkv * dk (norm 2); inv_freq: rot / 2 floats.
-PLLM_EXPORT int pllm_normed_qk_kv_write(int dtype, const void* proj, int row_stride, int k_off, int v_off, void* q_out,
-                                        const float* q_gain, const float* k_gain, int norm, float eps, float temp_coef,
-                                        int temp_every, const float* inv_freq, int rot, const int* positions, const int* slots,
-                                        void* kv_pool, int n_tokens, int nh, int nkv, int dk, int dv, int values_are_keys,
-                                        int page_size, long long pool_rows, int* status, cudaStream_t stream) {
+// proj: [tokens, row_stride] with q at 0, k at k_off (negative: queries only), v at v_off (ignored when values_are_keys, which
+// needs dv == dk).  Biases: float, one an entry, or null.  q_gain / k_gain: float, dk entries (norm 1) or nh * dk and nkv * dk
+// (norm 2), null for the others; inv_freq: rot / 2 floats.
+PLLM_EXPORT int pllm_normed_qk_kv_write(int dtype, const void* proj, int row_stride, int k_off, int v_off, const float* q_bias, const float* k_bias,
+                                        const float* v_bias, void* q_out, const float* q_gain, const float* k_gain, int norm, float eps,
+                                        float temp_coef, int temp_every, const float* inv_freq, int rot, int pairs, float rot_factor,
+                                        const int* positions, const int* slots, void* kv_pool, int n_tokens, int nh, int nkv, int dk, int dv,
+                                        int values_are_keys, int page_size, long long pool_rows, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return PLLM_OK;
     if (nh <= 0 || nkv <= 0 || dk <= 0 || dv <= 0 || page_size <= 0 || rot < 0 || rot > dk || rot % 2) return PLLM_ERR_SIZE;
-    if (norm < 0 || norm > 2 || (norm && (!q_gain || !k_gain)) || (rot && !inv_freq) || temp_every < 0) return PLLM_ERR_SIZE;
+    const bool gains = norm == 1 || norm == 2;
+    if (norm < 0 || norm > 3 || (gains && !q_gain) || (gains && k_off >= 0 && !k_gain) || (rot && !inv_freq) || temp_every < 0) return PLLM_ERR_SIZE;
     if (values_are_keys && dv != dk) return PLLM_ERR_SIZE;
-    const size_t smem = (size_t)(nh + nkv) * sizeof(float);
-    if (smem > 40 * 1024) return PLLM_ERR_LIMIT;
+    NormedQK a = {k_off, v_off, q_bias, k_bias, v_bias, gains ? q_gain : nullptr, gains ? k_gain : nullptr, norm, eps, temp_coef, temp_every,
+                  inv_freq, rot, pairs ? 1 : 0, rot_factor, nh, nkv, dk, dv, values_are_keys, page_size, pool_rows};
+    const size_t smem = ((size_t)nh * dk + (k_off >= 0 ? (size_t)nkv * dk : 0) + 8 + rot + nh + nkv) * sizeof(float);
+    if (smem > 200 * 1024) return PLLM_ERR_LIMIT;
     PLLM_DISPATCH_DTYPE(dtype, {
-        launch_chained(normed_qk_kv_write_kernel<T>, dim3(n_tokens), dim3(256), smem, stream, (const T*)proj, row_stride, k_off, v_off,
-                       (T*)q_out, q_gain, k_gain, norm, eps, temp_coef, temp_every, inv_freq, rot, positions, slots, (T*)kv_pool, nh,
-                       nkv, dk, dv, values_are_keys, page_size, pool_rows, status);
+        const bool quads = dk % 4 == 0 && dv % 4 == 0 && row_stride % 4 == 0 && (k_off < 0 || k_off % 4 == 0) && (values_are_keys || v_off % 4 == 0) &&
+                           (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)kv_pool) & (4 * sizeof(T) - 1)) == 0;
+        auto kernel = quads ? normed_qk_kv_write_kernel<T, 4> : normed_qk_kv_write_kernel<T, 1>;
+        if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        launch_chained(kernel, dim3(n_tokens), dim3(256), smem, stream, (const T*)proj, row_stride, a, (T*)q_out, positions, slots, (T*)kv_pool, status);
     });
     return launch_status();
 }

@@ -8,7 +8,8 @@
 //                       (the norm sits on the sublayer's OUTPUT a, the sum stays in float)
 //   sandwich_norm32     x[r] += norm(a[r] + bias) * gain_a, then y[i] = T(norm(x[r]) * gain): output norm, sum and input norm
 //   rmsnorm_from32      y[i] = T(x[r] / sqrt(mean(x[r]^2) + eps) * gain),  r = rows ? rows[i] : i
-//   embed_norm32        x[t] = e / sqrt(mean(e^2) + eps) * gain,  e = table[token[t]]       (a norm right behind the embedding)
+//   embed_norm32        x[t] = e / sqrt(mean(e^2) + eps) * gain + bias,  e = table[token[t]], its mean taken off first where
+//                       the norm is centered       (a norm right behind the embedding)
 //   add_scaled_norm32   x[r] += mult * d[r]  (d may be absent);  y[i] = T(x[r] / sqrt(mean(x[r]^2) + eps) * gain)
 //                       (the pre-norm block of a float stream whose sublayer outputs are multiplied by a constant;
 //                       with rows the sum is formed for those rows only and not stored)
@@ -243,8 +244,8 @@ PLLM_EXPORT int pllm_rmsnorm_from32(int dtype, const float* x, const float* gain
 // One CTA a token: the row is fetched once into registers-by-stride, its mean square reduced over the CTA.
 template <typename T>
 __global__ void __launch_bounds__(256) embed_norm32_kernel(const int* __restrict__ tokens, const T* __restrict__ table,
-                                                           const float* __restrict__ gain, float* __restrict__ out, int hidden,
-                                                           int vocab, float eps, int* status) {
+                                                           const float* __restrict__ gain, const float* __restrict__ bias, int centered,
+                                                           float* __restrict__ out, int hidden, int vocab, float eps, int* status) {
     __shared__ float scratch[32];
     pdl_launch_dependents();
     pdl_wait(KID_STREAM32);
@@ -253,22 +254,27 @@ __global__ void __launch_bounds__(256) embed_norm32_kernel(const int* __restrict
     const bool ok = tok >= 0 && tok < vocab;
     if (!ok && threadIdx.x == 0) atomicOr(status, 1);
     const T* src = table + (size_t)(ok ? tok : 0) * hidden;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) { const float v = to_f32(src[i]); ss += v * v; }
+    float mean = 0.f, ss = 0.f;
+    if (centered) {
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) mean += to_f32(src[i]);
+        mean = block_sum(mean, scratch) / (float)hidden;
+    }
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) { const float v = to_f32(src[i]) - mean; ss += v * v; }
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
     float* dst = out + (size_t)t * hidden;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = ok ? to_f32(src[i]) * inv * gain[i] : 0.f;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x)
+        dst[i] = ok ? (to_f32(src[i]) - mean) * inv * gain[i] + (bias ? bias[i] : 0.f) : 0.f;
 }
 
-PLLM_EXPORT int pllm_embed_norm32(int dtype, const int* tokens, const void* table, const float* gain, float* out, int n_tokens,
-                                  int hidden, int vocab, float eps, int* status, cudaStream_t stream) {
+PLLM_EXPORT int pllm_embed_norm32(int dtype, const int* tokens, const void* table, const float* gain, const float* bias, int centered,
+                                  float* out, int n_tokens, int hidden, int vocab, float eps, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return PLLM_OK;
     if (hidden <= 0 || vocab <= 0) return PLLM_ERR_SIZE;
     PLLM_DISPATCH_DTYPE(dtype, {
         const int threads = min(256, max(32, (hidden + 31) / 32 * 32));
-        launch_chained(embed_norm32_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream, tokens, (const T*)table, gain, out,
-                       hidden, vocab, eps, status);
+        launch_chained(embed_norm32_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream, tokens, (const T*)table, gain, bias,
+                       centered, out, hidden, vocab, eps, status);
     });
     return launch_status();
 }

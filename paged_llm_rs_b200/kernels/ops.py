@@ -88,7 +88,7 @@ def lib():
         sig["pllm_gemm_tcgen05_grouped"] = [P, P, P, c_int, c_int, c_int, c_int, c_float, P, c_int, P, P]
         sig["pllm_moe_pair_glu"] = [c_int, P, P, P, P] + [c_int] * 6 + [c_float, c_int, P, P]
         sig["pllm_moe_pair_down"] = [c_int, P, P, P, P, P, P, P] + [c_int] * 5 + [P, c_int, P]
-        sig["pllm_embed_norm32"] = [c_int, P, P, P, P, c_int, c_int, c_int, c_float, P, P]
+        sig["pllm_embed_norm32"] = [c_int, P, P, P, P, c_int, P, c_int, c_int, c_int, c_float, P, P]
         sig["pllm_add_scaled_norm32"] = [c_int, P, P, c_float, P, P, P, c_int, c_int, c_float, P]
         sig["pllm_add_scaled32"] = [c_int, P, P, c_float, c_ll, P]
         sig["pllm_scale32"] = [P, c_float, c_ll, P]
@@ -103,7 +103,8 @@ def lib():
         sig["pllm_sandwich_norm32"] = [c_int, P, P, P, P, P, P, P, c_int, c_int, c_float, P]
         sig["pllm_scaled_sum2"] = [c_int, P, P, c_float, c_float, P, c_ll, P]
         sig["pllm_swiglu_bias"] = [c_int, P, P, P, c_int, c_int, c_int, c_float, P]
-        sig["pllm_normed_qk_kv_write"] = [c_int, P, c_int, c_int, c_int, P, P, P, c_int, c_float, c_float, c_int, P, c_int, P, P, P] + [c_int] * 7 + [c_ll, P, P]
+        sig["pllm_normed_qk_kv_write"] = [c_int, P, c_int, c_int, c_int, P, P, P, P, P, P, c_int, c_float, c_float, c_int, P, c_int, c_int, c_float, P, P,
+                                          P] + [c_int] * 7 + [c_ll, P, P]
         sig["pllm_gate_mul"] = [c_int, P, P, c_int, c_int, c_int, c_int, c_int, P]
         sig["pllm_unary_act"] = [c_int, P, c_ll, c_int, P]
         sig["pllm_conv_rope_kv_write"] = [c_int, P, c_int, P, P, c_int, P, c_int, c_int, P, c_ll, P, c_int, P, P, P, P] + [c_int] * 6 + [c_ll, P, P]
@@ -118,7 +119,11 @@ def lib():
         sig["pllm_rope_table"] = [P, P, P, c_int, c_int, P]
         sig["pllm_linear_attention_mix"] = [c_int, P] + [c_int] * 5 + [c_float, c_float, c_int, P, P, P, P, P, P, c_int, c_float, P, P, c_int, c_int, P, c_ll,
                                             P, P, P] + [c_int] * 4 + [c_float, P]
-        wide = {"pllm_linear_attention_state_floats": [c_int] * 3, "pllm_linear_attention_scratch_floats": [c_int] * 6,
+        sig["pllm_add_terms_norm32"] = [c_int, P] + [P, c_int, c_float] * 3 + [P, P, c_int, P, P, c_int, c_int, c_float, P]
+        sig["pllm_channel_delta_mix"] = [c_int, P, c_int, P, P, c_int, c_int, P, c_int, P, P, c_int, P, c_int, P, P, P, c_int, c_int, P, c_ll, P, P, P,
+                                         P] + [c_int] * 6 + [c_float, P]
+        wide = {"pllm_channel_delta_state_floats": [c_int] * 5, "pllm_channel_delta_record_floats": [c_int] * 4,
+                "pllm_linear_attention_state_floats": [c_int] * 3, "pllm_linear_attention_scratch_floats": [c_int] * 6,
                 "pllm_mlstm_state_floats": [c_int] * 3, "pllm_delta_state_floats": [c_int] * 5}
         for name, args in wide.items():
             fn = getattr(L, name)
@@ -949,15 +954,16 @@ def moe_experts(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gu:
 # ---- a float32 stream with pre-norm blocks (csrc/stream32.cu) ----------------------------------------------------
 
 def embed_norm32(tokens: torch.Tensor, table: torch.Tensor, gain: torch.Tensor, eps: float, out: torch.Tensor,
-                 status: torch.Tensor) -> torch.Tensor:
-    """out[t] = rmsnorm(table[tokens[t]]) * gain as float32, whatever the table's dtype."""
-    _dev(tokens, table, gain, out, status)
-    _i32(tokens, "tokens"); _f32(out, "out"); _f32(gain, "gain")
+                 status: torch.Tensor, bias: Optional[torch.Tensor] = None, centered: bool = False) -> torch.Tensor:
+    """out[t] = norm(table[tokens[t]]) * gain (+ bias) as float32, whatever the table's dtype: over the root mean square or, with
+    ``centered``, the mean taken off first (a layer norm)."""
+    _dev(tokens, table, gain, bias, out, status)
+    _i32(tokens, "tokens"); _f32(out, "out"); _f32(gain, "gain"); _f32(bias, "bias")
     T, (V, H) = tokens.numel(), table.shape
-    if out.shape != (T, H) or gain.numel() != H:
-        raise KernelError(f"embed_norm32: out is {tuple(out.shape)}, expected {(T, H)}, with a gain of {H}")
-    _check(lib().pllm_embed_norm32(_code(table), _ptr(tokens), _ptr(table), _ptr(gain), _ptr(out), T, H, V, float(eps),
-                                   _ptr(status), _stream()), "embed_norm32")
+    if out.shape != (T, H) or gain.numel() != H or (bias is not None and bias.numel() != H):
+        raise KernelError(f"embed_norm32: out is {tuple(out.shape)}, expected {(T, H)}, with a gain (and bias) of {H}")
+    _check(lib().pllm_embed_norm32(_code(table), _ptr(tokens), _ptr(table), _ptr(gain), _ptr(bias), 1 if centered else 0, _ptr(out), T, H, V,
+                                   float(eps), _ptr(status), _stream()), "embed_norm32")
     return out
 
 
@@ -1182,45 +1188,56 @@ def scaled_sum2(x: torch.Tensor, y: torch.Tensor, a: float, b: float, out: Optio
 
 # ---- queries and keys that are normed before the attention, and a gate behind it (csrc/normed_qk.cu) ---------------------------
 
-QK_NORMS = {None: 0, "head": 1, "projection": 2}
+QK_NORMS = {None: 0, "head": 1, "projection": 2, "head_after_rotation": 3}
 
 
 def normed_qk_kv_write(proj: torch.Tensor, k_off: int, v_off: int, q_out: torch.Tensor, q_gain: Optional[torch.Tensor],
                        k_gain: Optional[torch.Tensor], norm: Optional[str], eps: float, temp_coef: float, temp_every: int,
                        inv_freq: Optional[torch.Tensor], rot: int, positions: torch.Tensor, slots: Optional[torch.Tensor],
                        kv_pool: Optional[torch.Tensor], num_heads: int, num_kv_heads: int, dk: int, dv: int, values_are_keys: bool,
-                       status: torch.Tensor) -> torch.Tensor:
-    """From a stacked projection ``proj`` [T, width] (q at 0, k at k_off, v at v_off) to the attention's inputs: q and k normed
-    (``norm``: None, "head": each head by its own root mean square with one gain of dk entries, "projection": all heads at
-    once with a gain of the projection's size), q times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) (temp_every 0:
-    not), both rotated on the first ``rot`` entries of each head; q to q_out [T, heads dk], k | v to row ``slots[t]`` of
-    kv_pool [pages, kv_heads, page_size, dk + dv].  ``values_are_keys``: v is the raw key projection (neither normed nor rotated)."""
-    _dev(proj, q_out, q_gain, k_gain, inv_freq, positions, slots, kv_pool, status)
-    _f32(q_gain, "q_gain"); _f32(k_gain, "k_gain"); _f32(inv_freq, "inv_freq"); _i32(positions, "positions"); _i32(slots, "slots")
+                       status: torch.Tensor, q_bias: Optional[torch.Tensor] = None, k_bias: Optional[torch.Tensor] = None,
+                       v_bias: Optional[torch.Tensor] = None, rot_pairs: bool = False, rot_factor: float = 1.0) -> torch.Tensor:
+    """From a stacked projection ``proj`` [T, width] (q at 0, k at k_off, v at v_off) to the attention's inputs: biases; q and k
+    normed (``norm``: None, "head": each head by its own root mean square with one gain of dk entries, "projection": all heads at
+    once with a gain of the projection's size, "head_after_rotation": each head by its root mean square behind the rotation, no
+    gain), q times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) (temp_every 0: not), both turned on the first ``rot`` entries
+    of each head (entry i with i + rot / 2, or with ``rot_pairs`` entry 2i with 2i + 1; cos and sin times ``rot_factor``); q to
+    q_out [T, heads dk], k | v to row ``slots[t]`` of kv_pool [pages, kv_heads, page_size, dk + dv].  ``values_are_keys``: v is
+    the raw key projection (neither normed nor rotated).  k_off negative: the projection holds queries only."""
+    _dev(proj, q_out, q_gain, k_gain, inv_freq, positions, slots, kv_pool, status, q_bias, k_bias, v_bias)
+    for t, n in ((q_gain, "q_gain"), (k_gain, "k_gain"), (inv_freq, "inv_freq"), (q_bias, "q_bias"), (k_bias, "k_bias"), (v_bias, "v_bias")):
+        _f32(t, n)
+    _i32(positions, "positions"); _i32(slots, "slots")
     T, width = proj.shape
+    keys = k_off >= 0
     if norm not in QK_NORMS:
         raise KernelError(f"normed_qk_kv_write: norm {norm!r} is not known; known: {list(QK_NORMS)}")
-    if k_off + num_kv_heads * dk > width or (not values_are_keys and v_off + num_kv_heads * dv > width) or num_heads * dk > width:
+    if num_heads * dk > width or (keys and (k_off + num_kv_heads * dk > width or (not values_are_keys and v_off + num_kv_heads * dv > width))):
         raise KernelError("normed_qk_kv_write: the projection is narrower than its parts")
     if q_out.numel() != T * num_heads * dk or q_out.dtype != proj.dtype:
         raise KernelError("normed_qk_kv_write: q_out does not fit")
-    n_gain = {None: (0, 0), "head": (dk, dk), "projection": (num_heads * dk, num_kv_heads * dk)}[norm]
-    if norm is not None and (q_gain is None or k_gain is None or q_gain.numel() != n_gain[0] or k_gain.numel() != n_gain[1]):
+    n_gain = {"head": (dk, dk), "projection": (num_heads * dk, num_kv_heads * dk)}.get(norm)
+    if n_gain is not None and (q_gain is None or q_gain.numel() != n_gain[0] or (keys and (k_gain is None or k_gain.numel() != n_gain[1]))):
         raise KernelError("normed_qk_kv_write: the gains do not fit the norm")
+    for t, n in ((q_bias, num_heads * dk), (k_bias, num_kv_heads * dk), (v_bias, num_kv_heads * dv)):
+        if t is not None and t.numel() != n:
+            raise KernelError("normed_qk_kv_write: one bias an entry of the projection")
     if rot and (inv_freq is None or inv_freq.numel() * 2 != rot):
         raise KernelError("normed_qk_kv_write: inv_freq must hold rot / 2 frequencies")
     if positions.numel() < T or (slots is not None and slots.numel() < T):
         raise KernelError("normed_qk_kv_write: positions / slots shorter than the tokens")
     page_size, pool_rows = 1, 0
     if kv_pool is not None:
+        if not keys:
+            raise KernelError("normed_qk_kv_write: a projection of queries only has nothing to store")
         if kv_pool.dim() != 4 or kv_pool.shape[1] != num_kv_heads or kv_pool.shape[3] != dk + dv or kv_pool.dtype != proj.dtype:
             raise KernelError(f"normed_qk_kv_write: the pool must be [pages, {num_kv_heads}, page_size, {dk + dv}] of {proj.dtype}")
         page_size, pool_rows = kv_pool.shape[2], kv_pool.shape[0] * kv_pool.shape[2]
-    _check(lib().pllm_normed_qk_kv_write(_code(proj), _ptr(proj), width, int(k_off), int(v_off), _ptr(q_out), _ptr(q_gain), _ptr(k_gain),
-                                         QK_NORMS[norm], float(eps), float(temp_coef), int(temp_every), _ptr(inv_freq), int(rot),
-                                         _ptr(positions), _ptr(slots), _ptr(kv_pool), T, num_heads, num_kv_heads, dk, dv,
-                                         1 if values_are_keys else 0, page_size, pool_rows, _ptr(status), _stream()),
-           "normed_qk_kv_write")
+    _check(lib().pllm_normed_qk_kv_write(_code(proj), _ptr(proj), width, int(k_off), int(v_off), _ptr(q_bias), _ptr(k_bias), _ptr(v_bias),
+                                         _ptr(q_out), _ptr(q_gain), _ptr(k_gain), QK_NORMS[norm], float(eps), float(temp_coef), int(temp_every),
+                                         _ptr(inv_freq), int(rot), 1 if rot_pairs else 0, float(rot_factor), _ptr(positions), _ptr(slots),
+                                         _ptr(kv_pool), T, num_heads, num_kv_heads, dk, dv, 1 if values_are_keys else 0, page_size, pool_rows,
+                                         _ptr(status), _stream()), "normed_qk_kv_write")
     return q_out
 
 
@@ -1314,6 +1331,56 @@ def delta_mix(u: torch.Tensor, conv_w: torch.Tensor, ba: torch.Tensor, a_log: to
                                 _ptr(segments), segments.shape[0], int(max_segment_tokens), _ptr(state), state.stride(0), _ptr(c_buf),
                                 _ptr(y_buf), _ptr(out), T, heads, kv_heads, dim, vdim, taps, float(eps), _stream()),
            "delta_mix", launches=3)
+    return out
+
+
+# ---- the gated delta rule with a decay a key entry (csrc/delta_rule.cu) --------------------------------------------------------
+
+def channel_delta_state_floats(heads: int, kv_heads: int, dim: int, vdim: int, taps: int) -> int:
+    """Floats of a request's state slot: every head's matrix, then each channel's last inputs in a ring of ``taps`` rows."""
+    return heads * dim * vdim + (taps * (2 * kv_heads * dim + heads * vdim) if taps > 1 else 0)
+
+
+def channel_delta_mix(u: torch.Tensor, conv_w: torch.Tensor, small: torch.Tensor, a1_off: int, a2: torch.Tensor, a_log: torch.Tensor,
+                      dt_bias: torch.Tensor, g1_off: int, g2: torch.Tensor, gain: torch.Tensor, segments: torch.Tensor,
+                      max_segment_tokens: int, state: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
+                      taps: int, eps: float, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """From a projection ``u`` [T, width] whose first columns are [q | k | v] (kv_heads dim, kv_heads dim, heads vdim) and a float32
+    projection ``small`` [T, width] (step sizes' logits in its first ``heads`` columns, the decays' short vector at a1_off) to the
+    output projection's input [T, heads vdim]: convolution and silu, unit q and k, decays exp(-exp(a_log) softplus(a2 a1 + dt_bias))
+    a key entry, the gated delta rule over each segment's tokens from and into its state slot, each head over its root mean square,
+    the gain (vdim entries, shared by the heads), sigmoid of the gate's logits.  These come as ``gate`` [T, heads vdim] in a step
+    with portions of prompts, and are formed as g2 times the short vector at column g1_off of ``u`` in one of decoded tokens
+    (max_segment_tokens 1)."""
+    _dev(u, conv_w, small, a2, a_log, dt_bias, g2, gain, segments, state, out, gate)
+    for t, n in ((small, "small"), (a_log, "a_log"), (dt_bias, "dt_bias"), (gain, "gain"), (state, "state")):
+        _f32(t, n)
+    _segments_ok(segments, "channel_delta_mix")
+    T, longest = u.shape[0], int(max_segment_tokens)
+    channels, rank, g_rank = 2 * kv_heads * dim + heads * vdim, a2.shape[1], g2.shape[1]
+    if u.shape[1] < channels or g1_off + g_rank > u.shape[1] or out.shape != (T, heads * vdim) or out.dtype != u.dtype:
+        raise KernelError("channel_delta_mix: u must hold q, k, v and the gate's short vector, out be [T, heads vdim], of one dtype")
+    if conv_w.shape != (channels, taps) or any(t.dtype != u.dtype for t in (conv_w, a2, g2)):
+        raise KernelError("channel_delta_mix: the convolution's taps must be [channels, taps], a2 and g2 matrices, of u's dtype")
+    if small.shape[0] != T or a1_off < heads or small.shape[1] < a1_off + rank or a2.shape[0] != heads * dim or g2.shape[0] != heads * vdim:
+        raise KernelError("channel_delta_mix: small, a2 or g2 does not fit")
+    if a_log.numel() != heads or dt_bias.numel() != heads * dim or gain.numel() != vdim:
+        raise KernelError("channel_delta_mix: one A_log a head, a dt_bias a key entry, and a gain of vdim entries")
+    if state.dim() != 2 or state.shape[1] < channel_delta_state_floats(heads, kv_heads, dim, vdim, taps):
+        raise KernelError("channel_delta_mix: the state slots are too small")
+    records = v_buf = y_buf = None
+    launches = 1
+    if longest != 1:
+        if gate is None or gate.shape != out.shape or gate.dtype != u.dtype:
+            raise KernelError("channel_delta_mix: a step with portions of prompts needs the gate's logits, [T, heads vdim] of u's dtype")
+        records = torch.empty(int(lib().pllm_channel_delta_record_floats(T, segments.shape[0], heads, dim)), dtype=torch.float32, device=u.device)
+        v_buf = torch.empty((T, heads * vdim), dtype=torch.float32, device=u.device)
+        y_buf = torch.zeros((T, heads * vdim), dtype=torch.float32, device=u.device)     # (rows of no segment stay zero)
+        launches = 3
+    _check(lib().pllm_channel_delta_mix(
+        _code(u), _ptr(u), u.shape[1], _ptr(conv_w), _ptr(small), small.shape[1], int(a1_off), _ptr(a2), rank, _ptr(a_log), _ptr(dt_bias), int(g1_off),
+        _ptr(g2), g_rank, _ptr(gate), _ptr(gain), _ptr(segments), segments.shape[0], longest, _ptr(state), state.stride(0), _ptr(records), _ptr(v_buf),
+        _ptr(y_buf), _ptr(out), T, heads, kv_heads, dim, vdim, taps, float(eps), _stream()), "channel_delta_mix", launches=launches)
     return out
 
 
@@ -1503,6 +1570,27 @@ def gated_sum_norm32(x: torch.Tensor, gain: torch.Tensor, out: torch.Tensor, eps
         _ptr(mixed_bias), _ptr(fed), strides[3], _ptr(fed_gate), strides[4], _ptr(fed_bias), _ptr(embedded), _ptr(vector), _ptr(x_out), _ptr(gain),
         _ptr(out), _ptr(shift), _ptr(shifted), _ptr(gain2), _ptr(out2), _ptr(segments), segments.shape[0] if segments is not None else 0,
         _ptr(state), state.stride(0) if state is not None else 0, _ptr(rows), n, W, float(eps), _stream()), "gated_sum_norm32")
+    return out
+
+
+def add_terms_norm32(x: torch.Tensor, terms, gain: torch.Tensor, eps: float, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
+                     centered: bool = False, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x (float32, in place) += the sum of constant * tensor over ``terms`` (at most three (tensor, constant); a tensor may be a
+    column range of a wider one); out[i] = norm(x[r]) gain (+ bias), r = rows[i] or i: over the root mean square or, with
+    ``centered``, the mean taken off first (a layer norm).  With ``rows`` the sum is formed for those rows only and x stays as it
+    is."""
+    _dev(x, gain, bias, out, rows)
+    _f32(x, "x"); _f32(gain, "gain"); _f32(bias, "bias"); _i32(rows, "rows")
+    T, W = x.shape
+    n = rows.numel() if rows is not None else T
+    if len(terms) > 3 or out.shape != (n, W) or gain.numel() != W or (bias is not None and bias.numel() != W):
+        raise KernelError("add_terms_norm32: three terms at most; out must be [rows, width], gain and bias of the stream's width")
+    args = []
+    for i in range(3):
+        t, c = terms[i] if i < len(terms) else (None, 0.0)
+        args += [_ptr(t), _cols(t, (T, W), out.dtype, "add_terms_norm32: a term"), float(c)]
+    _check(lib().pllm_add_terms_norm32(_code(out), _ptr(x), *args, _ptr(gain), _ptr(bias), 1 if centered else 0, _ptr(out), _ptr(rows), n, W, float(eps),
+                                       _stream()), "add_terms_norm32")
     return out
 
 

@@ -4,3 +4,4 @@ from . import bumisun  # registers Bumisun
 from . import pamarax  # registers Pamarax
 from . import tebozen  # registers Tebozen
 from . import reperax  # registers Reperax
+from . import tubevik  # registers Tubevik

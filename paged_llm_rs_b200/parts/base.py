@@ -274,6 +274,16 @@ class Part:
         return f"{self.prefix}.{leaf}" if self.prefix else leaf
 
 
+def stack_rows(matrices, multiple: int = 8) -> torch.Tensor:
+    """Matrices that read the same input as one, its rows filled up with zeros to a multiple of ``multiple`` (so that the rows of
+    its product start on vector boundaries)."""
+    rows = sum(m.shape[0] for m in matrices)
+    more = -rows % multiple
+    if more:
+        matrices = list(matrices) + [matrices[0].new_zeros((more, matrices[0].shape[1]))]
+    return torch.cat(matrices, 0).contiguous()
+
+
 class Norm(Part):
     def forward(self, x: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         raise NotImplementedError

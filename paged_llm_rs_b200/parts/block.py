@@ -170,7 +170,29 @@ class SideBySideGatedStreamBlock(Block):
         return stream, out
 
 
+class SideBySideStreamBlock(Block):
+    """x + m (mixer(norm(x)) + ff(norm(x))) on a float32 stream: both sublayers read ONE norm of x.  Its norm is a
+    ``TermsStreamNorm`` named "mixer", which holds the model's constant m.  A layer may have no feed-forward.  What is handed on
+    beside the stream is what is pending: the mixer's terms (two mixers side by side give one each) and the feed-forward's
+    output, with their constants; ONE kernel adds them and norms the sum."""
+
+    def forward(self, stream, pending, step, cache, writes_cache=True):
+        rt, norm = self.mixer.rt, self.norms["mixer"]
+        h = norm.add_norm(stream, pending)
+        if hasattr(self.mixer, "forward_terms"):
+            terms = list(self.mixer.forward_terms(h, step, cache, writes_cache))
+        else:
+            terms = [(self.mixer.forward(h, step, cache, writes_cache), 1.0)]
+        if self.feed_forward is not None:
+            terms.append((self.feed_forward.forward(h, step), 1.0))
+        pending = [(t, norm.mult * c) for t, c in terms]
+        if rt.trace is not None and self.prefix:
+            rt.record(f"{self.prefix}.out", norm.settled(stream, pending))
+        return stream, pending
+
+
 register_block("side_by_side_gated_stream32", SideBySideGatedStreamBlock)
+register_block("side_by_side_stream32", SideBySideStreamBlock)
 register_block("prenorm_residual", PreNormResidualBlock)
 register_block("prenorm_stream32", PreNormStreamBlock)
 register_block("outnorm_residual", OutputNormResidualBlock)

@@ -48,28 +48,30 @@ class TokenEmbedding(Part):
 
 
 class NormedTokenEmbedding(Part):
-    """A row gather with an RMS norm right behind it, into a float32 residual stream: x = norm(table[token]) * gain.
-    ``norm`` names the gain's tensor."""
+    """A row gather with a norm right behind it, into a float32 residual stream: x = norm(table[token]) * gain, an RMS norm or,
+    with ``centered``, a layer norm with a bias.  ``norm`` names the gain's tensor, ``norm`` and ".b" the bias's."""
 
     def __init__(self, spec, rt):
         super().__init__(spec, rt)
         p = spec.params
         self.vocab, self.hidden, self.eps = int(p["vocab_size"]), int(p["hidden_size"]), float(p["eps"])
-        self.leaf, self.norm_name = p.get("leaf", "weight"), p["norm"]
-        self.table = self.gain = None
+        self.leaf, self.norm_name, self.centered = p.get("leaf", "weight"), p["norm"], bool(p.get("centered", False))
+        self.table = self.gain = self.bias = None
 
     def _table_name(self):
         return self._name(self.leaf) if self.leaf else self.prefix
 
     def tensors(self):
-        return [TensorSpec(self._table_name(), (self.vocab, self.hidden)), TensorSpec(self.norm_name, (self.hidden,), "gain")]
+        return [TensorSpec(self._table_name(), (self.vocab, self.hidden)), TensorSpec(self.norm_name, (self.hidden,), "gain")] + (
+            [TensorSpec(self.norm_name + ".b", (self.hidden,), "offset")] if self.centered else [])
 
     def bind(self, tensors):
         self.table, self.gain = tensors[self._table_name()], tensors[self.norm_name]
+        self.bias = tensors[self.norm_name + ".b"] if self.centered else None
 
     def forward(self, tokens: torch.Tensor) -> torch.Tensor:
         out = torch.empty((tokens.numel(), self.hidden), dtype=torch.float32, device=self.table.device)
-        ops.embed_norm32(tokens, self.table, self.gain, self.eps, out, self.rt.status)
+        ops.embed_norm32(tokens, self.table, self.gain, self.eps, out, self.rt.status, bias=self.bias, centered=self.centered)
         self.rt.record(self._name("out"), out)
         return out
 

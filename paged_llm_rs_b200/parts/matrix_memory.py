@@ -19,6 +19,14 @@ request).  With h the mixer's input, S a head's matrix (key entries by value ent
     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q          (o is read after the update)
     out = W_o (o / rms(o) a head * gain * silu(W_g h))                     gain: vdim entries, shared by the heads
 
+``channel_gated_delta_rule``: the same with a decay a key entry and a gate behind a product in two factors,
+
+    g = exp(-exp(A_log of the head) softplus(W_a2 (W_a1 h) + dt_bias))      one a key entry of every head, acting on S's rows
+    out = W_o (o / rms(o) a head * gain * sigmoid(W_g2 (W_g1 h)))
+
+(W_a1 h leaves its product in float32, the second product of the decays is formed in float32 beside the recurrence; how many
+entries W_a1 h and W_g1 h have only the file knows).
+
 The gates' and step sizes' projections leave in float32; everything from there to the output projection's input is
 float32 whatever the compute dtype.  A step's requests are found through its segment list on the device, so a captured
 step replays with any requests; the slot also keeps each convolution channel's last taps - 1 inputs.
@@ -28,9 +36,12 @@ from __future__ import annotations
 
 import torch
 
+from ..errors import WeightError
 from ..kernels import ops
-from .base import Mixer, StateNeed, register_mixer
+from .base import Mixer, StateNeed, register_mixer, stack_rows
 from .spec import TensorSpec
+
+RANDOM_RANK = 16        # the inner size of a product in two factors in a model of random weights
 
 
 class MatrixLSTM(Mixer):
@@ -129,5 +140,56 @@ class GatedDeltaRule(Mixer):
         return out
 
 
+class ChannelGatedDeltaRule(GatedDeltaRule):
+    def __init__(self, spec, rt, position_encodings=None):
+        super().__init__(spec, rt, position_encodings)
+        for k in ("a1", "a2", "g1", "g2"):
+            self.names.setdefault(k, k)
+        self.w_small = self.w_a2 = self.w_g2 = None
+        self.g1_off = 2 * self.kv_heads * self.dim + self.heads * self.vdim
+        self.rank = self.g_rank = 0
+
+    def tensors(self):
+        n, W, H, R = self.names, self.hidden, self.heads, RANDOM_RANK
+        own = {self._name(n["g"]), self._name(n["a"]), self._name(n["dt_bias"])}
+        qk, v = H * self.dim, H * self.vdim
+        return [t for t in super().tensors() if t.name not in own] + [
+            TensorSpec(self._name(n["dt_bias"]), (qk,), "offset"), TensorSpec(self._name(n["a1"]), (None, W), drawn=(R, W)),
+            TensorSpec(self._name(n["a2"]), (qk, None), drawn=(qk, R)), TensorSpec(self._name(n["g1"]), (None, W), drawn=(R, W)),
+            TensorSpec(self._name(n["g2"]), (v, None), drawn=(v, R))]
+
+    def bind(self, tensors):
+        t = lambda k: tensors[self._name(self.names[k])]
+        self.w_in, self.w_small = stack_rows([t("q"), t("k"), t("v"), t("g1")]), stack_rows([t("b"), t("a1")])
+        self.conv_w = torch.cat([t("q_conv"), t("k_conv"), t("v_conv")], 0).contiguous()
+        self.w_a2, self.w_g2 = t("a2").contiguous(), t("g2").contiguous()
+        self.w_o, self.gain, self.a_log, self.dt_bias = t("o"), t("norm"), t("a_log"), t("dt_bias")
+        for one, two in (("a1", "a2"), ("g1", "g2")):
+            if t(one).shape[0] != t(two).shape[1]:
+                raise WeightError(f"{self._name(self.names[one])} has {t(one).shape[0]} rows, {self._name(self.names[two])} {t(two).shape[1]} columns")
+        self.rank, self.g_rank = t("a1").shape[0], t("g1").shape[0]
+
+    def cache_need(self):
+        return StateNeed((ops.channel_delta_state_floats(self.heads, self.kv_heads, self.dim, self.vdim, self.taps),), torch.float32)
+
+    def forward(self, x, step, cache, writes_cache=True):
+        st = self.rt.status
+        u = ops.linear(x, self.w_in, status=st)
+        small = ops.linear(x, self.w_small, out_dtype=torch.float32, status=st)
+        longest = step.max_segment_tokens or step.n_tokens
+        gate = None
+        if longest != 1:
+            gate = ops.linear(u[:, self.g1_off:self.g1_off + self.g_rank].contiguous(), self.w_g2, status=st)
+        y = torch.empty((x.shape[0], self.heads * self.vdim), dtype=x.dtype, device=x.device)
+        ops.channel_delta_mix(u, self.conv_w, small, self.heads, self.w_a2, self.a_log, self.dt_bias, self.g1_off, self.w_g2, self.gain,
+                              step.segments, longest, cache, y, self.heads, self.kv_heads, self.dim, self.vdim, self.taps, self.eps, gate=gate)
+        out = ops.linear(y, self.w_o, status=st)
+        if self.rt.trace is not None:
+            for leaf, t in (("in.out", u), ("small", small), ("o.in", y), ("out", out)):
+                self.rt.record(self._name(leaf), t)
+        return out
+
+
+register_mixer("channel_gated_delta_rule", ChannelGatedDeltaRule)
 register_mixer("matrix_lstm", MatrixLSTM)
 register_mixer("gated_delta_rule", GatedDeltaRule)

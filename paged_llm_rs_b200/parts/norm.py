@@ -180,6 +180,44 @@ class PendingGated:
         return a
 
 
+class TermsStreamNorm(RMSNorm):
+    """A norm in a decoder whose residual stream stays float32 and whose sublayers read ONE norm of it: what is pending is a list
+    of (output, constant), three at most, which ``add_norm`` adds into the stream (in place) and whose sum it norms into the
+    compute dtype, in one kernel.  ``centered``: a layer norm with a bias (named by the gain's name and ".b"), else an RMS norm.
+    ``mult``: the constant on all that the block's sublayers give."""
+
+    def __init__(self, spec, rt):
+        super().__init__(spec, rt)
+        self.mult, self.centered = float(spec.params.get("mult", 1.0)), bool(spec.params.get("centered", False))
+        self.bias = None
+
+    def tensors(self):
+        return super().tensors() + ([TensorSpec(self._gain_name() + ".b", (self.width,), "offset")] if self.centered else [])
+
+    def bind(self, tensors):
+        super().bind(tensors)
+        self.bias = tensors[self._gain_name() + ".b"] if self.centered else None
+
+    def forward(self, x, rows=None):
+        return self.add_norm(x, None, rows)
+
+    def add_norm(self, residual, delta, rows=None):
+        if residual.dtype != torch.float32:
+            raise ValueError("the residual stream of this norm is float32")
+        n = rows.numel() if rows is not None else residual.shape[0]
+        out = torch.empty((n, self.width), dtype=self.rt.dtype, device=residual.device)
+        ops.add_terms_norm32(residual, delta or [], self.gain, self.eps, out, bias=self.bias, centered=self.centered, rows=rows)
+        self.rt.record(self._name("out"), out)
+        return out
+
+    def settled(self, stream, delta):
+        """The stream with all that is pending added, as a tensor of its own."""
+        x = stream.clone()
+        ops.add_terms_norm32(x, delta, self.gain, self.eps, torch.empty(x.shape, dtype=self.rt.dtype, device=x.device), bias=self.bias,
+                             centered=self.centered)
+        return x
+
+
 class GatedStreamRMSNorm(RMSNorm):
     """RMSNorm in a decoder whose residual stream stays float32 and whose sublayers sit side by side behind gates: its block
     runs two of them, the token shift and the pending sum in one kernel; alone (the model's last norm) ``add_norm`` forms the
@@ -219,6 +257,7 @@ class GatedStreamRMSNorm(RMSNorm):
 
 register_norm("rmsnorm", RMSNorm)
 register_norm("rmsnorm_gated_stream32", GatedStreamRMSNorm)
+register_norm("terms_stream32", TermsStreamNorm)
 register_norm("rmsnorm_stream32", StreamRMSNorm)
 register_norm("rmsnorm_scaled_stream32", ScaledStreamRMSNorm)
 register_norm("rmsnorm_sandwich_stream32", SandwichStreamRMSNorm)

@@ -15,6 +15,22 @@ import torch
 from .base import PositionEncoding, register_position_encoding
 
 
+def rotary_frequencies(dims: int, base: float, scaling=None):
+    """(frequencies of the dims / 2 pairs in float64, factor on cos and sin): base^(-2i / dims) and 1, or with ``scaling``
+    (factor, original, fast, slow) the YaRN blend of them: a pair that turns more than ``fast`` times within ``original``
+    positions keeps its frequency, one that turns fewer than ``slow`` times has it divided by ``factor``, those between go
+    linearly from one to the other; cos and sin are then multiplied by 0.1 ln(factor) + 1."""
+    i = np.arange(dims // 2, dtype=np.float64)
+    f = np.power(np.float64(base), -2.0 * i / dims)
+    if scaling is None:
+        return f, 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+    pair = lambda turns: dims * np.log(original / (2.0 * np.pi * float(turns))) / (2.0 * np.log(float(base)))
+    lo, hi = max(np.floor(pair(scaling["fast"])), 0.0), min(np.ceil(pair(scaling["slow"])), dims - 1.0)
+    ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
+    return f / factor * ramp + f * (1.0 - ramp), float(0.1 * np.log(factor) + 1.0)
+
+
 class RotaryEncoding(PositionEncoding):
     def __init__(self, spec, rt):
         super().__init__(spec, rt)
