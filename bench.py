@@ -1378,6 +1378,217 @@ def reperax_kernels(z, pk):
     return out
 
 
+# ---- the windowed-attention / chunked-attention-beside-delta-rule decoder (Tubevik) ----------------------------------------
+# Sizes that resemble real layers, at the widths of the 0.6B and of a 2B-class shape: windowed attention (1024 tokens, capped
+# scores, a gate a head, YaRN rotation of half of each head) of sixteen heads over eight kv heads of 128, every second such layer
+# borrowing the keys and values of the one before; beside chunked attention (1024) with values of 64, the delta rule of width / 128
+# heads of 128 x 128 over half as many q/k heads with a decay of inner size 64 (a random model's) behind convolutions of four taps; a clamped gated
+# feed-forward.  The other model is Pamarax at the same width, depth, head sizes, feed-forward and vocabulary: its attention layers
+# and its side-by-side layers (attention over the whole context, gated delta rule) in turn.
+TUBEVIK_SIZES = {
+    "1024": dict(width=1024, heads=16, kv_heads=8, dim=128, vdim=128, window=1024, rot=64, left_vdim=64, chunk=1024, d_heads=8, d_kv_heads=4,
+                 d_dim=128, d_vdim=128, conv=4, rank=64, ff=3072),
+    "2048": dict(width=2048, heads=16, kv_heads=8, dim=128, vdim=128, window=1024, rot=64, left_vdim=64, chunk=1024, d_heads=16, d_kv_heads=8,
+                 d_dim=128, d_vdim=128, conv=4, rank=64, ff=6144),
+}
+
+
+def tubevik_config(z, layers):
+    att = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["vdim"], scale=z["dim"] ** -0.5, softcap=30.0, mask=dict(size=z["window"]),
+               rot=dict(dims=z["rot"], base=500000.0, scaling=dict(factor=8.0, original=8192, fast=32.0, slow=1.0)))
+    left = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["left_vdim"], scale=z["dim"] ** -0.5, mask=dict(size=z["chunk"]),
+                rot=dict(dims=z["rot"], base=10000.0))
+    right = dict(heads=z["d_heads"], kv_heads=z["d_kv_heads"], dim=z["d_dim"], vdim=z["d_vdim"], conv=z["conv"])
+    par = dict(type="parallel", mixer=dict(left=left, right=right, left_scale=0.8, right_scale=0.6))
+    out = []
+    for i in range(layers):
+        mixer = par if i % 2 else dict(type="attention", mixer=dict(att, kv_from=i - 2) if i % 4 == 2 else att)
+        out.append(dict(mixer, mlp=dict(kind="dense", ff=z["ff"], limit=7.0)))
+    return dict(architecture="Tubevik", vocab=LATENT_VOCAB, width=z["width"], norm=dict(eps=1e-6), residual_mult=0.5, logit_softcap=30.0, layers=out)
+
+
+def tubevik_beside_matrix(size, layers, pk, clocks, steps, warmup, which="both", kernels_only=False):
+    """Decode (batch 1, 8, 64 at context 4096) and the 2048-token prefill of the Tubevik shape ``size`` and of the Pamarax shape
+    of the same width, layers, head sizes, feed-forward and vocabulary: tokens a second, side by side; then Tubevik's own
+    kernels alone beside the like kernels of Pamarax."""
+    import gc
+    import torch
+    from paged_llm_rs_b200 import Engine, write_random_model
+
+    z = TUBEVIK_SIZES[size]
+    mz = MATRIX_SIZES[size]
+    matrix = matrix_config(mz, 4)
+    matrix["layers"] = [matrix["layers"][2 * (i % 2)] for i in range(layers)]        # attention, side by side, ...
+    out = dict(size=size, layers=layers, vocab=LATENT_VOCAB, tubevik=dict(z))
+    for name, cfg in () if kernels_only else (("tubevik", tubevik_config(z, layers)), ("pamarax", matrix)):
+        if which not in ("both", name):
+            continue
+        tmp = tempfile.mkdtemp(prefix="pllm_bench_", dir=scratch_dir())
+        try:
+            model_dir = write_random_model(os.path.join(tmp, "model"), cfg, 0, device="cuda")
+            ctx = 4096
+            pages = 64 * (ctx // PAGE + 4) + (PREFILL_TOKENS + 1024) // PAGE + 64
+            eng = Engine(model_dir, dtype="bfloat16", block_size=PAGE, blocks=pages, max_batch=64, chunk=PREFILL_TOKENS,
+                         prefix_cache=False)
+            shutil.rmtree(tmp, ignore_errors=True)
+            runner = eng.runner
+            for g in runner.cache.groups:
+                if g.pool is not None:
+                    g.pool.normal_(0.0, 1.0)
+            res = dict(weight_bytes=runner.weight_bytes(), cache_bytes_a_token=runner.cache.bytes_per_token())
+            for b in (1, 8, 64):
+                ms, launches, spread = decode_point(runner, b, ctx, max(5, steps // 2), warmup, clocks, repeats=4)
+                res[f"decode_b{b}_tok_s"] = round(b / (spread["median_ms"] / 1e3), 1)
+                res[f"decode_b{b}_ms"] = spread["median_ms"]
+                res[f"decode_b{b}_launches"] = launches
+            pms, _ = prefill_point(runner, LATENT_VOCAB, clocks, repeats=4)
+            res["prefill_ms"] = round(pms, 3)
+            res["prefill_tok_s"] = round(PREFILL_TOKENS / (pms / 1e3), 1)
+            out[name] = res
+            del eng, runner
+        finally:
+            shutil.rmtree(tmp, ignore_errors=True)
+            gc.collect()
+            torch.cuda.empty_cache()
+    out["kernels"] = tubevik_kernels(z, pk)
+    like = matrix_kernels(mz, pk)
+    out["kernels"].update({f"pamarax_{k}": v for k, v in like.items() if not k.startswith("mlstm")})
+    return out
+
+
+def tubevik_kernels(z, pk):
+    """Tubevik's own kernels alone, at the sizes of ``z``, each beside its like kernel of another design where that is not among
+    Pamarax's: device time (CUDA events, the median of nine after three warm-ups, an L2 flush before each), the algorithmic
+    bytes and FLOPs, and the fraction of the measured copy bandwidth or bfloat16 product rate they come to."""
+    import numpy as np
+    import torch
+    from paged_llm_rs_b200.kernels import attention_plan, ops
+    from paged_llm_rs_b200.parts.base import AttentionWork
+
+    dev, bf = "cuda", torch.bfloat16
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    target = 2 * ops.sm_count()
+    out = {}
+
+    def timed(fn):
+        for _ in range(3):
+            fn()
+        torch.cuda.synchronize()
+        ts = []
+        for _ in range(9):
+            flush_l2()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record(); fn(); b.record()
+            torch.cuda.synchronize()
+            ts.append(a.elapsed_time(b))
+        return statistics.median(ts)
+
+    def note(name, ms, nbytes, flops):
+        r = dict(us=round(ms * 1e3, 2), mbytes=round(nbytes / 1e6, 2), gflop=round(flops / 1e9, 3),
+                 hbm_frac=round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 4),
+                 bf16_frac=round(flops / (ms / 1e3) / 1e12 / pk["bf16_tflops"], 4))
+        r["frac_of_slower_bound"] = round(max(r["hbm_frac"], r["bf16_frac"]), 4)
+        out[name] = r
+
+    def plan(segs, tile, ctas, window=0, chunk=0):
+        work, red, parts = attention_plan.plan_attention(segs, tile, window, ctas, target, chunk=chunk)
+        wd = torch.from_numpy(np.ascontiguousarray(work)).reshape(-1, 8).to(dev)
+        rd = torch.from_numpy(np.ascontiguousarray(red)).reshape(-1, 4).to(dev) if len(red) else torch.zeros(1, 4, dtype=torch.int32, device=dev)
+        singles = all(n == 1 for _, n, _ in segs)
+        return lambda heads, hd: AttentionWork(wd, torch.tensor([len(work)], dtype=torch.int32, device=dev), len(work), rd,
+                                                torch.tensor([len(red)], dtype=torch.int32, device=dev), len(red),
+                                                torch.zeros(max(parts, 1), heads, hd, device=dev), torch.zeros(max(parts, 1), heads, 2, device=dev),
+                                                kinds=1 if singles else 2, many_splits=attention_plan.many_splits(len(segs), ctas, target))
+
+    ctx, B, T, W = 4096, 64, PREFILL_TOKENS, z["width"]
+    n_pages = B * ctx // PAGE
+    tables = torch.randperm(n_pages, dtype=torch.int32).view(B, ctx // PAGE).to(dev)
+    cases = {"decode_b64_ctx4096": [(i, 1, ctx - 1) for i in range(B)], "prefill_2048": [(0, T, 0)]}
+    nh, nkv, dk = z["heads"], z["kv_heads"], z["dim"]
+    inv = torch.rand(z["rot"] // 2, device=dev)
+    # -- the two attentions, each beside the same kernel without what it adds (cap; the one more, chunks instead of a window)
+    for label, dv, variants in (("window", z["vdim"], [("attention_window_capped", z["window"], 0, 30.0, False), ("like_attention_window", z["window"], 0, 0.0, False)]),
+                                ("chunk", z["left_vdim"], [("attention_chunk_extra_one", 0, z["chunk"], 0.0, True), ("like_attention_window_64", z["chunk"], 0, 0.0, False)])):
+        pool = torch.randn(n_pages, nkv, PAGE, dk + dv, device=dev).to(bf)
+        tile, ctas = ops.attention_sink_tile_tokens(nh, nkv, bf, dk, dv), ops.attention_sink_ctas_per_item(nh, nkv, bf, dk, dv)
+        for case, segs in cases.items():
+            n = sum(c for _, c, _ in segs)
+            q, o = torch.randn(n, nh * dk, device=dev).to(bf), torch.empty(n, nh * dv, dtype=bf, device=dev)
+            for name, win, ch, cap, one in variants:
+                seen = lambda p: p % ch + 1 if ch else min(p + 1, win)
+                keys = sum(seen(p + i) for _, c, p in segs for i in range(c))
+                seg_keys = sum((p + c) - (p - p % ch if ch else max(0, p - win + 1)) for _, c, p in segs)
+                w = plan(segs, tile, ctas, win, ch)(nh, dv)
+                sinks = torch.zeros(nh, device=dev) if one else None
+                ms = timed(lambda: ops.attention_sink(q, pool, tables, w, o, sinks, nh, nkv, dk, dv, win, 0, dk ** -0.5, cap, status, chunk=ch))
+                note(f"{name}_{case}", ms, seg_keys * nkv * (dk + dv) * 2 + n * nh * (dk + dv) * 2, 2 * nh * (dk + dv) * keys)
+            # what stands between the projection and the attention
+            k_off, v_off = nh * dk, (nh + nkv) * dk
+            width = v_off + nkv * dv + (nh if label == "window" else 0)
+            proj = torch.randn(n, width, device=dev).to(bf)
+            pos = torch.arange(n, dtype=torch.int32, device=dev)
+            slots = torch.randperm(n_pages * PAGE, dtype=torch.int32)[:n].to(dev)
+            ones = lambda k: torch.ones(k, device=dev)
+            if label == "window":
+                gq, gk, bq, bk, bv = ones(nh * dk), ones(nkv * dk), ones(nh * dk), ones(nkv * dk), ones(nkv * dv)
+                run = lambda: ops.normed_qk_kv_write(proj, k_off, v_off, q, gq, gk, "projection", 1e-6, 0.0, 0, inv, z["rot"], pos, slots, pool, nh, nkv,
+                                                     dk, dv, False, status, q_bias=bq, k_bias=bk, v_bias=bv, rot_factor=1.2)
+                note(f"normed_qk_kv_write_biases_projection_{case}", timed(run), 2 * (v_off + nkv * dv) * n * 2, 0)
+                wq, zero = proj[:, :nh * dk].contiguous(), None
+                run = lambda: ops.normed_qk_kv_write(wq, -1, 0, q, gq, zero, "projection", 1e-6, 0.0, 0, inv, z["rot"], pos, slots, zero, nh, nkv,
+                                                     dk, dv, False, status, q_bias=bq, rot_factor=1.2)
+                note(f"normed_qk_queries_only_{case}", timed(run), 2 * nh * dk * n * 2, 0)
+                note(f"gate_mul_a_head_{case}", timed(lambda: ops.gate_mul(o, proj[:, v_off + nkv * dv:], "sigmoid", per=dv)), n * nh * (2 * dv + 1) * 2, 0)
+                wide = torch.randn(n, nh * dv, device=dev).to(bf)
+                note(f"like_gate_mul_an_entry_{case}", timed(lambda: ops.gate_mul(o, wide, "sigmoid")), n * nh * 3 * dv * 2, 0)
+            else:
+                run = lambda: ops.normed_qk_kv_write(proj, k_off, v_off, q, None, None, "head_after_rotation", 1e-6, 0.0, 0, inv, z["rot"], pos, slots, pool,
+                                                     nh, nkv, dk, dv, False, status, rot_pairs=True)
+                note(f"normed_qk_kv_write_pairs_then_norm_{case}", timed(run), 2 * proj.numel() * 2, 0)
+        del pool
+    # -- the delta rule between its projections
+    H, G, d, E, taps, R = z["d_heads"], z["d_kv_heads"], z["d_dim"], z["d_vdim"], z["conv"], z["rank"]
+    ch = 2 * G * d + H * E
+    floats = ops.channel_delta_state_floats(H, G, d, E, taps)
+    state = torch.zeros(B + 1, floats, device=dev)
+    cw, gain = torch.randn(ch, taps, device=dev).to(bf), torch.ones(E, device=dev)
+    a2, g2 = (torch.randn(H * d, R, device=dev) * 0.1).to(bf), (torch.randn(H * E, R, device=dev) * 0.1).to(bf)
+    a_log, dt = torch.zeros(H, device=dev), torch.zeros(H * d, device=dev)
+    for case, segs in cases.items():
+        n = sum(c for _, c, _ in segs)
+        u = torch.randn(n, ch + R, device=dev).to(bf)
+        small = torch.randn(n, H + R, device=dev)
+        sg = torch.tensor([(t0, c, p, i + 1) for i, (t0, c, p) in enumerate(segs)], dtype=torch.int32, device=dev)
+        y = torch.empty(n, H * E, dtype=bf, device=dev)
+        longest = max(c for _, c, _ in segs)
+        gate = torch.randn(n, H * E, device=dev).to(bf) if longest != 1 else None
+        ms = timed(lambda: ops.channel_delta_mix(u, cw, small, H, a2, a_log, dt, ch, g2, gain, sg, longest, state, y, H, G, d, E, taps, 1e-6, gate=gate))
+        # (counted as for the like recurrence: projection read twice, convolved channels and read-out in float written and read once, gate, state)
+        note(f"channel_delta_mix_{case}", ms, n * (ch + H * E) * 2 * 2 + n * ch * 4 * 2 + small.numel() * 4 + n * H * E * 4 * 2 + y.numel() * 2 + len(segs) * floats * 4 * 2,
+             8 * n * H * d * E)
+    del state
+    # -- the sum of three terms with the layer norm; the layer norm behind the embedding; the clamped activation; the logits' cap
+    ff = z["ff"]
+    table = torch.randn(LATENT_VOCAB, W, device=dev).to(bf)
+    w_gu = (torch.randn(2 * ff, W, device=dev) * 0.02).to(bf)
+    for case, n in (("decode_b64", B), ("prefill_2048", T)):
+        x, vec = torch.randn(n, W, device=dev), torch.ones(W, device=dev)
+        a1, a2_, f, y = (torch.randn(n, W, device=dev).to(bf) for _ in range(4))
+        note(f"add_terms_norm32_{case}", timed(lambda: ops.add_terms_norm32(x, [(a1, 0.4), (a2_, 0.3), (f, 0.5)], vec, 1e-6, y, bias=vec, centered=True)),
+             n * W * (4 + 4 + 3 * 2 + 2), 0)
+        toks = torch.randint(0, LATENT_VOCAB, (n,), device=dev, dtype=torch.int32)
+        note(f"embed_norm32_centered_{case}", timed(lambda: ops.embed_norm32(toks, table, vec, 1e-6, x, status, bias=vec, centered=True)), n * W * (2 + 4), 0)
+        note(f"like_embed_norm32_{case}", timed(lambda: ops.embed_norm32(toks, table, vec, 1e-6, x, status)), n * W * (2 + 4), 0)
+        h = torch.randn(n, W, device=dev).to(bf)
+        nbytes, flops = w_gu.numel() * 2 + n * (W + ff) * 2, 2 * n * 2 * ff * W
+        note(f"gate_up_clamped_{case}", timed(lambda: ops.linear_glu(h, w_gu, status=status, act="clamped", limit=7.0)), nbytes, flops)
+        note(f"like_gate_up_silu_{case}", timed(lambda: ops.linear_glu(h, w_gu, status=status)), nbytes, flops)
+    logits = torch.randn(B, LATENT_VOCAB, device=dev)
+    note("softcap32_decode_b64", timed(lambda: ops.softcap32(logits, 30.0)), logits.numel() * 8, 0)
+    note("like_scale32_decode_b64", timed(lambda: ops.scale32(logits, 1.0)), logits.numel() * 8, 0)
+    return out
+
+
 TRACE_KERNELS = {0: "(tcgen05 kernel)", 1: "embed", 2: "rmsnorm", 3: "swiglu", 4: "qk_norm_rope_kv", 5: "attention_generic", 6: "attention_reduce",
                  7: "attention_mma", 8: "attention_tma", 9: "skinny_gemm", 10: "sample_partial", 11: "sample_final", 12: "gemm_tcgen05", 13: "attention_tcgen05"}
 TRACE_FILES = ["elementwise", "qk_norm_rope_kv", "attention_generic", "attention_mma", "attention_decode_tma", "sampling",
@@ -1544,8 +1755,12 @@ def main(argv=None) -> int:
     ap.add_argument("--reperax-size", choices=sorted(REPERAX_SIZES), default="1024",
                     help="with --only reperax: the width of the retention / chunked-attention-beside-gated-linear-attention decoder (Reperax)")
     ap.add_argument("--reperax-model", choices=["both", "reperax", "pamarax"], default="both", help="with --only reperax: one model alone")
+    ap.add_argument("--tubevik-size", choices=sorted(TUBEVIK_SIZES), default="1024",
+                    help="with --only tubevik: the width of the windowed-attention / chunked-attention-beside-delta-rule decoder (Tubevik)")
+    ap.add_argument("--tubevik-model", choices=["both", "tubevik", "pamarax", "kernels"], default="both",
+                    help="with --only tubevik: one model alone, or the kernels alone")
     ap.add_argument("--only", choices=["decode", "prefill", "long-prompt", "timeline", "reference-kernel", "plain-cpu", "latent", "hybrid", "matrix",
-                                       "tebozen", "reperax"],
+                                       "tebozen", "reperax", "tubevik"],
                     default=None,
                     help="run one part alone and print a short line (for profiling; not a bench record); "
                          "long-prompt: a prompt of --context tokens in portions of 2048, each portion timed; "
@@ -1561,7 +1776,9 @@ def main(argv=None) -> int:
                          "tebozen: the same for the decoder of differential attention, matrix LSTM and latent attention layers with "
                          "squared-relu experts (Tebozen) beside the Bumisun shape of equal size (--tebozen-size, --layers, default 8); "
                          "reperax: the same for the decoder of retention layers and chunked attention beside gated linear attention "
-                         "(Reperax) beside the Pamarax shape of equal size (--reperax-size, --layers, default 8)")
+                         "(Reperax) beside the Pamarax shape of equal size (--reperax-size, --layers, default 8); "
+                         "tubevik: the same for the decoder of windowed attention over lent keys and chunked attention beside a delta "
+                         "rule with a decay a key entry (Tubevik) beside the Pamarax shape of equal size (--tubevik-size, --layers, default 8)")
     args = ap.parse_args(argv)
 
     if args.impl == "reference":
@@ -1615,6 +1832,13 @@ def main(argv=None) -> int:
     if args.only == "reperax":
         clocks.start()
         out = reperax_beside_matrix(args.reperax_size, args.layers or 8, pk, clocks, steps, warmup, which=args.reperax_model)
+        out["clocks"] = clocks.stop()
+        print(json.dumps(out))
+        return 0
+    if args.only == "tubevik":
+        clocks.start()
+        out = tubevik_beside_matrix(args.tubevik_size, args.layers or 8, pk, clocks, steps, warmup, which=args.tubevik_model,
+                                    kernels_only=args.tubevik_model == "kernels")
         out["clocks"] = clocks.stop()
         print(json.dumps(out))
         return 0

@@ -82,9 +82,10 @@ __device__ __forceinline__ float dr_dot(const T* __restrict__ row, const float* 
 __host__ __device__ __forceinline__ int dr_block_floats(int dp) { return 13 * dp + 36; }
 __host__ __device__ __forceinline__ int dr_record_floats(int dp) { return DR_RUN / DR_BLOCK * dr_block_floats(dp); }
 
-// grid (runs of the step's segments, heads), 128 threads.  small: [tokens, small_stride] float, b_raw at 0 (H), a1 at a1_off.
+// grid (runs of the step's segments, heads), 128 threads.  The scan behind it is not let in early: its CTAs would crowd onto the SMs
+// that this kernel leaves first.  small: [tokens, small_stride] float, b_raw at 0 (H), a1 at a1_off.
 template <typename T>
-__global__ void __launch_bounds__(128) delta_prepare_kernel(const T* u, DRShape sh, const T* __restrict__ conv_w, const float* small, int small_stride,
+__global__ void __launch_bounds__(128, 5) delta_prepare_kernel(const T* u, DRShape sh, const T* __restrict__ conv_w, const float* small, int small_stride,
                                                             int a1_off, const T* __restrict__ a2, int rank, const float* __restrict__ a_log,
                                                             const float* __restrict__ dt_bias, const MMSegment* __restrict__ segs, int n_segs,
                                                             const float* state, float* __restrict__ records, float* __restrict__ v_buf) {
@@ -94,7 +95,7 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const T* u, DRShape 
     float* k_s = q_s + DR_RUN * dp;
     float* g_s = k_s + DR_RUN * dp;
     float* a1_s = g_s + DR_RUN * dp;         // [DR_RUN][padded]
-    pdl_launch_dependents();
+    float* x_s = a1_s + DR_RUN * padded;     // [DR_RUN + taps - 1][128] the convolution's inputs, a channel a thread
     const MMBlock b = mm_find_block(segs, n_segs, blockIdx.x, DR_RUN);
     if (b.seg < 0) return;
     const MMSegment s = segs[b.seg];
@@ -109,35 +110,63 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const T* u, DRShape 
         const int t = i / padded, r = i - t * padded;
         a1_s[i] = (t < nt && r < rank) ? small[(size_t)(s.first + t0 + t) * small_stride + a1_off + r] : 0.f;
     }
-    __syncthreads();
-    // the convolutions: a thread has one channel's inputs of the run in registers
-    for (int it = tid; it < 2 * d + E; it += blockDim.x) {
-        const int ch = it < d ? kh * d + it : it < 2 * d ? sh.G * d + kh * d + (it - d) : 2 * sh.G * d + h * E + (it - 2 * d);
-        float w[DR_MAX_TAPS], x[DR_RUN + DR_MAX_TAPS - 1];
+    // the convolutions, 128 channels at a time: q's and k's of the kv head, then v's of the head
+    const int rows = DR_RUN + sh.taps - 1, chans = 2 * d + E;
+    auto channel = [&](int it) { return it < d ? kh * d + it : it < 2 * d ? sh.G * d + kh * d + (it - d) : 2 * sh.G * d + h * E + (it - 2 * d); };
+    constexpr int V = Vec16<T>::N;
+    const bool vec = d % V == 0 && E % V == 0 && sh.u_stride % V == 0 && (reinterpret_cast<uintptr_t>(u) & 15) == 0;
+    for (int c0 = 0; c0 < chans; c0 += 128) {
+        __syncthreads();
+        if (vec) {
+#pragma unroll 4
+            for (int i = tid; i < rows * (128 / V); i += 128) {
+                const int j = i / (128 / V), it = c0 + i % (128 / V) * V, r = t0 + j - (sh.taps - 1);
+                float f[V];
+                if (it >= chans || r >= t0 + nt) {
 #pragma unroll
-        for (int j = 0; j < DR_MAX_TAPS; j++) w[j] = j < sh.taps ? to_f32(conv_w[(size_t)ch * sh.taps + j]) : 0.f;
+                    for (int k = 0; k < V; k++) f[k] = 0.f;
+                } else if (r >= 0) {
+                    Vec16<T> v;
+                    v.load(u + (size_t)(s.first + r) * sh.u_stride + channel(it));
+                    v.unpack(f);
+                } else {
 #pragma unroll
-        for (int j = 0; j < DR_RUN + DR_MAX_TAPS - 1; j++) {
-            const int t = j - (sh.taps - 1);
-            x[j] = (j < DR_RUN + sh.taps - 1 && t < nt) ? dr_input(u, sh, s, ring, t0 + t, ch) : 0.f;
+                    for (int k = 0; k < V; k++) f[k] = dr_input(u, sh, s, ring, r, channel(it) + k);
+                }
+#pragma unroll
+                for (int k = 0; k < V; k += 4) *reinterpret_cast<float4*>(x_s + j * 128 + it - c0 + k) = make_float4(f[k], f[k + 1], f[k + 2], f[k + 3]);
+            }
+        } else {
+#pragma unroll 4
+            for (int j = 0; j < rows; j++) {
+                const int it = c0 + tid, r = t0 + j - (sh.taps - 1);
+                x_s[j * 128 + tid] = (it < chans && r < t0 + nt) ? dr_input(u, sh, s, ring, r, channel(it)) : 0.f;
+            }
+        }
+        __syncthreads();
+        const int it = c0 + tid;
+        if (it >= chans) continue;
+        const T* wr = conv_w + (size_t)channel(it) * sh.taps;
+        float acc[DR_RUN];
+#pragma unroll
+        for (int t = 0; t < DR_RUN; t++) acc[t] = 0.f;
+        for (int j = 0; j < sh.taps; j++) {
+            const float w = to_f32(wr[j]);
+#pragma unroll
+            for (int t = 0; t < DR_RUN; t++) acc[t] = fmaf(w, x_s[(t + j) * 128 + tid], acc[t]);
         }
         float* dst = it < d ? q_s + it : k_s + (it - d);
 #pragma unroll
         for (int t = 0; t < DR_RUN; t++) {
-            float acc = 0.f;
-#pragma unroll
-            for (int j = 0; j < DR_MAX_TAPS; j++) {
-                if (j >= sh.taps) break;
-                acc = fmaf(w[j], x[t + j], acc);
-            }
-            if (t >= nt) continue;
-            const float c = mm_silu(acc);
+            if (t >= nt) break;
+            const float c = mm_silu(acc[t]);
             if (it < 2 * d) dst[t * dp] = c;
             else v_buf[((size_t)(s.first + t0 + t) * sh.H + h) * E + (it - 2 * d)] = c;
         }
     }
     // the decays: a thread has one key entry, its row of a2 in registers 16 entries at a time
     const float rate = -expf(a_log[h]);
+    const bool vec_a = rank % V == 0 && (reinterpret_cast<uintptr_t>(a2) & 15) == 0;
     for (int n = tid; n < d; n += blockDim.x) {
         const float bias = dt_bias[h * d + n];
         float z[DR_RUN];
@@ -147,7 +176,16 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(const T* u, DRShape 
         for (int r0 = 0; r0 < rank; r0 += 16) {
             float w[16];
 #pragma unroll
-            for (int r = 0; r < 16; r++) w[r] = r0 + r < rank ? to_f32(row[r0 + r]) : 0.f;
+            for (int r = 0; r < 16; r++) w[r] = !vec_a && r0 + r < rank ? to_f32(row[r0 + r]) : 0.f;
+            if (vec_a) {
+#pragma unroll
+                for (int r = 0; r < 16; r += V) {
+                    if (r0 + r >= rank) break;
+                    Vec16<T> v;
+                    v.load(row + r0 + r);
+                    v.unpack(w + r);
+                }
+            }
 #pragma unroll
             for (int t = 0; t < DR_RUN; t++) {
                 const float4* a4 = reinterpret_cast<const float4*>(a1_s + t * padded + r0);
@@ -263,14 +301,15 @@ __device__ __forceinline__ void dr_meet(float (&val)[16], int part) {
     }
 }
 
-// grid (segments, heads, slices of e).  Thread (columns p0 + 2 cg, p0 + 2 cg + 1; part): rows (j PARTS + part) 4 ... + 3, j < NQ.
-template <typename T, int PARTS, int NQ>
-__global__ void __launch_bounds__(256) delta_blocks_kernel(const T* u, DRShape sh, const float* records, const float* v_buf,
+// grid (segments, heads, slices of e).  u is read for the convolution's last inputs only (bf16: its dtype).  Thread (columns p0 + 2 cg, p0 + 2 cg + 1; part): rows (j PARTS + part) 4 ... + 3, j < NQ.
+template <int PARTS, int NQ>
+__global__ void __launch_bounds__(256, 1) delta_blocks_kernel(const void* u, int is_bf16, DRShape sh, const float* records, const float* v_buf,
                                                            const MMSegment* __restrict__ segs, int n_segs, float* state,
                                                            float* __restrict__ y, int Ps) {
     extern __shared__ __align__(16) float dr_smem[];
     constexpr int R = PARTS >= 16 ? 1 : 16 / PARTS;
-    const int H = sh.H, d = sh.d, E = sh.E, dp = sh.dp, RB = dr_block_floats(dp), RR = dr_record_floats(dp);
+    constexpr int dp = PARTS * NQ * 4, RB = 13 * dp + 36, RR = DR_RUN / DR_BLOCK * RB;        // (dr_padded, dr_block_floats, dr_record_floats)
+    const int H = sh.H, d = sh.d, E = sh.E;
     const int STAGE = RR + DR_RUN * Ps;              // a record, then the run's values [16][Ps]
     pdl_launch_dependents();
     const MMSegment s = segs[blockIdx.x];
@@ -300,6 +339,8 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const T* u, DRShape s
             st[c][2 * j + 1] = mm_pair(x[2], x[3]);
         }
     const int runs = (s.count + DR_RUN - 1) / DR_RUN;
+    // where this lane's read-outs go: sums x = PARTS == 32 ? part / 2 : part * R + r, of which those from eight on are of queries
+    float* yo = y + ((size_t)s.first * H + h) * E + e;
     auto fetch = [&](int run) {
         float* dst = dr_smem + (run & 1) * STAGE;
         const float* src = records + ((size_t)(first_run + run) * H + h) * RR;
@@ -391,8 +432,9 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const T* u, DRShape s
                 float o = val[r];
                 o = fmaf(c ? uu[0][1] : uu[0][0], m.x, o); o = fmaf(c ? uu[1][1] : uu[1][0], m.y, o);
                 o = fmaf(c ? uu[2][1] : uu[2][0], m.z, o); o = fmaf(c ? uu[3][1] : uu[3][0], m.w, o);
-                if (t0 + i < nt && cl + c < Ps && e + c < E) y[((size_t)(s.first + run * DR_RUN + t0 + i) * H + h) * E + e + c] = o;
+                if (t0 + i < nt && cl + c < Ps && e + c < E) yo[i * H * E + c] = o;
             }
+            yo += (size_t)DR_BLOCK * H * E;
         }
     }
 #pragma unroll
@@ -414,7 +456,8 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const T* u, DRShape s
     for (int i = tid; i < nv + extra; i += blockDim.x) {
         const int ch = i < nv ? 2 * sh.G * d + h * E + p0 + i : i < nv + d ? kh * d + (i - nv) : sh.G * d + kh * d + (i - nv - d);
         for (int r = max(0, s.count - (sh.taps - 1)); r < s.count; r++)
-            ring[(size_t)((s.before + r) % sh.taps) * sh.channels + ch] = to_f32(u[(size_t)(s.first + r) * sh.u_stride + ch]);
+            ring[(size_t)((s.before + r) % sh.taps) * sh.channels + ch] =
+                is_bf16 ? to_f32(((const bf16*)u)[(size_t)(s.first + r) * sh.u_stride + ch]) : ((const float*)u)[(size_t)(s.first + r) * sh.u_stride + ch];
     }
 }
 
@@ -422,6 +465,7 @@ __global__ void __launch_bounds__(256) delta_blocks_kernel(const T* u, DRShape s
 // rows, group, group + groups, ...  Ps: columns a slice (256 / (Ps / VEC) groups).  Every segment has one token at most.
 // g1: [tokens, u_stride] at g1_off of the projection, the gate's short vector; g2 [H e, g_rank].
 #define DR_STEP_THREADS 256
+#define DR_STEP_ROWS 16          // rows a thread, where eight slices allow it (eight rows in twice the CTAs: 46 us against 31 at 64 requests of 8 x 128 x 128)
 template <typename T, int VEC, int NR>
 __global__ void __launch_bounds__(DR_STEP_THREADS, NR * VEC <= 64 ? 2 : 1) delta_step_kernel(
     const T* u, DRShape sh, const T* __restrict__ conv_w, const float* small, int small_stride, int a1_off, const T* __restrict__ a2, int rank,
@@ -438,7 +482,8 @@ __global__ void __launch_bounds__(DR_STEP_THREADS, NR * VEC <= 64 ? 2 : 1) delta
     float* k_s = q_s + d;                      // [d]
     float* d_s = k_s + d;                      // [d] decays
     float* v_s = d_s + d;                      // [Ps] values, then what is written
-    float* p_s = v_s + Ps;                     // [2][groups][Ps] shares of the products with key and query
+    float* z_s = v_s + Ps;                     // [Ps] gates
+    float* p_s = z_s + Ps;                     // [2][groups][Ps] shares of the products with key and query
     pdl_launch_dependents();
     const MMSegment s = segs[blockIdx.x];
     if (s.count <= 0) return;                  // (a head's slices share the segment: the whole cluster leaves)
@@ -460,6 +505,11 @@ __global__ void __launch_bounds__(DR_STEP_THREADS, NR * VEC <= 64 ? 2 : 1) delta
             st[r][0] = in ? S[(size_t)n * E + e] : 0.f;
         }
     }
+    // the weights' rows do not come from the kernels before either
+    for (int i = tid; i < d + Ps; i += DR_STEP_THREADS) {
+        const char* row = i < d ? (const char*)(a2 + (size_t)(h * d + i) * rank) : (const char*)(g2 + (size_t)(h * E + min(p0 + i - d, E - 1)) * g_rank);
+        for (int o = 0; o < (i < d ? rank : g_rank) * (int)sizeof(T); o += 128) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(row + o));
+    }
     pdl_wait(KID_DELTA_RULE);
     const size_t tok = s.first;
     for (int r = tid; r < rank; r += DR_STEP_THREADS) a1_s[r] = small[tok * small_stride + a1_off + r];
@@ -470,6 +520,7 @@ __global__ void __launch_bounds__(DR_STEP_THREADS, NR * VEC <= 64 ? 2 : 1) delta
         if (c >= 0 && p0 + c >= E) { v_s[c] = 0.f; continue; }
         const int ch = i < d ? kh * d + i : i < 2 * d ? sh.G * d + kh * d + (i - d) : 2 * sh.G * d + h * E + p0 + c;
         float acc = 0.f;
+#pragma unroll 4
         for (int j = 0; j < sh.taps; j++)
             acc = fmaf(to_f32(conv_w[(size_t)ch * sh.taps + j]), dr_input(u, sh, s, ring, j - (sh.taps - 1), ch), acc);
         acc = mm_silu(acc);
@@ -480,10 +531,15 @@ __global__ void __launch_bounds__(DR_STEP_THREADS, NR * VEC <= 64 ? 2 : 1) delta
     __syncthreads();
     const float rate = -expf(a_log[h]);
     const bool vec_a = rank % Vec16<T>::N == 0 && (reinterpret_cast<uintptr_t>(a2) & 15) == 0;
+    const bool vec_g = g_rank % Vec16<T>::N == 0 && (reinterpret_cast<uintptr_t>(g2) & 15) == 0;
     float sq = 0.f, sk = 0.f, kq = 0.f;
-    for (int n = tid; n < d; n += DR_STEP_THREADS) {
-        d_s[n] = expf(rate * mm_softplus(dr_dot(a2 + (size_t)(h * d + n) * rank, a1_s, rank, vec_a) + dt_bias[h * d + n]));
-        const float a = q_s[n], b = k_s[n];
+    for (int i = tid; i < d + Ps; i += DR_STEP_THREADS) {
+        if (i >= d) {
+            if (p0 + i - d < E) z_s[i - d] = mm_sigmoid(dr_dot(g2 + (size_t)(h * E + p0 + i - d) * g_rank, g1_s, g_rank, vec_g));
+            continue;
+        }
+        d_s[i] = expf(rate * mm_softplus(dr_dot(a2 + (size_t)(h * d + i) * rank, a1_s, rank, vec_a) + dt_bias[h * d + i]));
+        const float a = q_s[i], b = k_s[i];
         sq = fmaf(a, a, sq); sk = fmaf(b, b, sk); kq = fmaf(a, b, kq);
     }
     sq = warp_sum(sq); sk = warp_sum(sk); kq = warp_sum(kq);
@@ -545,10 +601,6 @@ __global__ void __launch_bounds__(DR_STEP_THREADS, NR * VEC <= 64 ? 2 : 1) delta
     ss = 0.f;
 #pragma unroll
     for (int w = 0; w < DR_STEP_THREADS / 32; w++) ss += scratch[0][w];
-    float gate = 0.f;
-    const bool mine = tid < Ps && p0 + tid < E;
-    const bool vec_g = g_rank % Vec16<T>::N == 0 && (reinterpret_cast<uintptr_t>(g2) & 15) == 0;
-    if (mine) gate = mm_sigmoid(dr_dot(g2 + (size_t)(h * E + p0 + tid) * g_rank, g1_s, g_rank, vec_g));
     if (gridDim.y > 1) {
         cg::cluster_group cluster = cg::this_cluster();
         if (tid == 0) slice_ss = ss;
@@ -557,7 +609,7 @@ __global__ void __launch_bounds__(DR_STEP_THREADS, NR * VEC <= 64 ? 2 : 1) delta
         for (int r = 0; r < (int)gridDim.y; r++) ss += *cluster.map_shared_rank(&slice_ss, r);       // in the order of the slices
         cluster.sync();                        // (nobody leaves while its sum may still be read)
     }
-    if (mine) out[tok * H * E + (size_t)h * E + p0 + tid] = from_f32<T>(o / sqrtf(ss / (float)E + eps) * gain[p0 + tid] * gate);
+    if (tid < Ps && p0 + tid < E) out[tok * H * E + (size_t)h * E + p0 + tid] = from_f32<T>(o / sqrtf(ss / (float)E + eps) * gain[p0 + tid] * z_s[tid]);
 }
 
 // PARTS lanes a column and NQ quads of rows a lane: as many lanes as there are quads, up to a warp.
@@ -614,10 +666,10 @@ PLLM_EXPORT int pllm_channel_delta_mix(int dtype, const void* u, int u_stride, c
         while (Ps * slices < E) Ps *= 2;
         if (Ps < VEC) Ps = VEC;
         auto rows = [&]() { const int groups = DR_STEP_THREADS / (Ps / VEC); return groups > 0 ? (d + groups - 1) / groups : d; };
-        while (slices < 8 && Ps > VEC && (Ps > DR_STEP_THREADS || rows() > 16)) { slices *= 2; Ps /= 2; }
+        while (slices < 8 && Ps > VEC && (Ps > DR_STEP_THREADS || rows() > DR_STEP_ROWS)) { slices *= 2; Ps /= 2; }
         if (Ps > DR_STEP_THREADS || rows() > 32) return PLLM_ERR_LIMIT;
         const int groups = DR_STEP_THREADS / (Ps / VEC), nr = rows();
-        const size_t smem = ((size_t)(rank + 3) / 4 * 4 + (g_rank + 3) / 4 * 4 + 3 * d + Ps + 2 * (size_t)groups * Ps) * sizeof(float);
+        const size_t smem = ((size_t)(rank + 3) / 4 * 4 + (g_rank + 3) / 4 * 4 + 3 * d + 2 * Ps + 2 * (size_t)groups * Ps) * sizeof(float);
         if (smem > 200 * 1024) return PLLM_ERR_LIMIT;
         PLLM_DISPATCH_DTYPE(dtype, {
 #define DR_STEP(V, N) do { \
@@ -641,19 +693,21 @@ PLLM_EXPORT int pllm_channel_delta_mix(int dtype, const void* u, int u_stride, c
         warps /= 2;
     const int Ps = warps * per_warp, slices = (E + Ps - 1) / Ps;
     const size_t smem = 2 * (size_t)(dr_record_floats(sh.dp) + DR_RUN * Ps) * sizeof(float);
-    const size_t psmem = ((size_t)3 * DR_RUN * sh.dp + (size_t)DR_RUN * ((rank + 15) / 16 * 16)) * sizeof(float);
+    const size_t psmem = ((size_t)3 * DR_RUN * sh.dp + (size_t)DR_RUN * ((rank + 15) / 16 * 16) + (size_t)(DR_RUN + taps - 1) * 128) * sizeof(float);
     if (smem > 225 * 1024 || psmem > 225 * 1024) return PLLM_ERR_LIMIT;
     PLLM_DISPATCH_DTYPE(dtype, {
         if (psmem > 48 * 1024) cudaFuncSetAttribute(delta_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)psmem);
         launch_chained(delta_prepare_kernel<T>, dim3(n_segs + n_tokens / DR_RUN, H), dim3(128), psmem, stream, (const T*)u, sh, (const T*)conv_w, small,
                        small_stride, a1_off, (const T*)a2, rank, a_log, dt_bias, sg, n_segs, (const float*)state, records, v_buf);
+    });
 #define DR_SCAN(P, Q) do { \
-            if (smem > 48 * 1024) cudaFuncSetAttribute(delta_blocks_kernel<T, P, Q>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-            launch_chained(delta_blocks_kernel<T, P, Q>, dim3(n_segs, H, slices), dim3(warps * 32), smem, stream, (const T*)u, sh, \
-                           (const float*)records, (const float*)v_buf, sg, n_segs, state, y_buf, Ps); } while (0)
-        if (parts == 1) DR_SCAN(1, 1); else if (parts == 2) DR_SCAN(2, 1); else if (parts == 4) DR_SCAN(4, 1);
-        else if (parts == 8) DR_SCAN(8, 1); else if (parts == 16) DR_SCAN(16, 1);
-        else if (nq == 1) DR_SCAN(32, 1); else if (nq == 2) DR_SCAN(32, 2); else DR_SCAN(32, 4);
+        if (smem > 48 * 1024) cudaFuncSetAttribute(delta_blocks_kernel<P, Q>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        launch_chained(delta_blocks_kernel<P, Q>, dim3(n_segs, H, slices), dim3(warps * 32), smem, stream, u, dtype == PLLM_BF16 ? 1 : 0, sh, \
+                       (const float*)records, (const float*)v_buf, sg, n_segs, state, y_buf, Ps); } while (0)
+    if (parts == 1) DR_SCAN(1, 1); else if (parts == 2) DR_SCAN(2, 1); else if (parts == 4) DR_SCAN(4, 1);
+    else if (parts == 8) DR_SCAN(8, 1); else if (parts == 16) DR_SCAN(16, 1);
+    else if (nq == 1) DR_SCAN(32, 1); else if (nq == 2) DR_SCAN(32, 2); else DR_SCAN(32, 4);
+    PLLM_DISPATCH_DTYPE(dtype, {
         launch_head_norm_gate<T>(y_buf, nullptr, gate, H * E, gain, out, n_tokens, H, E, 0, 0, eps, stream);
     });
     return launch_status();

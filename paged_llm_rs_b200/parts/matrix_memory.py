@@ -41,7 +41,7 @@ from ..kernels import ops
 from .base import Mixer, StateNeed, register_mixer, stack_rows
 from .spec import TensorSpec
 
-RANDOM_RANK = 16        # the inner size of a product in two factors in a model of random weights
+RANDOM_RANK = 64        # the inner size of a product in two factors in a model of random weights
 
 
 class MatrixLSTM(Mixer):
