@@ -196,7 +196,7 @@ def kernel_delta(dtype, H, G, d, e, taps, cuts, pad, seed, ranks=(6, 4), rate=-2
     (4, 2, 16, 24, 3, (6, 4), [(1, 0), (1, 5), (1, 300)], 2),                                 # decoded tokens
     (3, 3, 20, 12, 1, (1, 9), [(1, 9), (1, 0)], 0), (2, 1, 20, 37, 16, (24, 8), [(1, 3), (1, 40)], 1),
     (1, 1, 256, 256, 4, (16, 32), [(1, 77)], 0), (2, 2, 512, 24, 2, (8, 1), [(1, 7)], 0), (4, 1, 4, 300, 5, (3, 3), [(1, 3), (1, 1)], 0),
-    (2, 1, 1, 1, 2, (1, 1), [(1, 4), (1, 0)], 0), (6, 6, 32, 32, 4, (24, 24), [(1, i) for i in range(40)], 24),
+    (2, 1, 1, 1, 2, (1, 1), [(1, 4), (1, 0)], 0), (5, 5, 32, 28, 4, (20, 12), [(1, i) for i in range(40)], 24),
     (1, 1, 384, 512, 2, (4, 4), [(1, 5)], 0), (8, 4, 128, 128, 4, (128, 128), [(1, 9)] * 3, 1),
     (4, 2, 16, 24, 3, (6, 4), [(5, 0), (1, 5), (33, 2), (2, 0)], 3),                          # portions beside decoded tokens
     (1, 1, 32, 32, 4, (16, 8), [(70, 0), (1, 6), (19, 40), (16, 0), (17, 3), (4, 4), (3, 1)], 2),
